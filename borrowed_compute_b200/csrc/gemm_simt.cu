@@ -7,10 +7,11 @@
 // share the launch, because each thread walks k in order on its own.
 //
 // Epilogues: store in the operand type; store as float (scores); add into a float buffer
-// (the residual stream); SwiGLU over a weight that stacks gate rows on up rows.
+// (the residual stream); SwiGLU over a weight that stacks gate rows on up rows; the square of relu; xIELU with its two
+// numbers; floats whose first columns are gated by their own sigmoid.
 #include "common.cuh"
 
-enum { EPI_STORE = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_RELU2 = 4 };
+enum { EPI_STORE = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_RELU2 = 4, EPI_XIELU = 5, EPI_SILU_F32 = 6 };
 
 #define BM 64
 #define BN 64
@@ -53,7 +54,7 @@ __device__ __forceinline__ void load_tile(const T* __restrict__ src, int rows, i
 
 template <class T, int EPI, bool VEC>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ X, const T* __restrict__ W, T* __restrict__ out_act,
-                                                        float* __restrict__ out_f32, int M, int N, int K) {
+                                                        float* __restrict__ out_f32, int M, int N, int K, float act_a, float act_b, int act_cols) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Bs[BK][BN + 4];
     __shared__ float Cs[EPI == EPI_SWIGLU ? BK : 1][BN + 4];
@@ -105,6 +106,14 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ X,
                 const float z = fmaxf(acc[i][j], 0.0f);
                 out_act[o] = from_f32<T>(z * z);
             }
+            if (EPI == EPI_XIELU) {
+                const float z = acc[i][j];
+                out_act[o] = from_f32<T>(fmaf(0.5f, z, z > 0.0f ? act_a * z * z : act_b * (expm1f(z) - z)));
+            }
+            if (EPI == EPI_SILU_F32) {
+                const float z = acc[i][j];
+                out_f32[o] = n < act_cols ? z / (1.0f + expf(-z)) : z;
+            }
             if (EPI == EPI_STORE_F32) out_f32[o] = acc[i][j];
             if (EPI == EPI_ADD_F32) out_f32[o] += acc[i][j];
             if (EPI == EPI_SWIGLU) {
@@ -116,39 +125,50 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ X,
 }
 
 template <class T, int EPI>
-static int launch(const void* X, const void* W, void* out, int M, int N, int K, cudaStream_t s) {
+static int launch(const void* X, const void* W, void* out, int M, int N, int K, float a, float b, int cols, cudaStream_t s) {
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
     const bool vec = K % 4 == 0 && ((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0);
-    T* oa = (EPI == EPI_STORE || EPI == EPI_SWIGLU || EPI == EPI_RELU2) ? (T*)out : nullptr;
-    float* of = (EPI == EPI_STORE_F32 || EPI == EPI_ADD_F32) ? (float*)out : nullptr;
+    T* oa = (EPI == EPI_STORE || EPI == EPI_SWIGLU || EPI == EPI_RELU2 || EPI == EPI_XIELU) ? (T*)out : nullptr;
+    float* of = (EPI == EPI_STORE_F32 || EPI == EPI_ADD_F32 || EPI == EPI_SILU_F32) ? (float*)out : nullptr;
     if (vec)
-        bc_launch(gemm_simt_kernel<T, EPI, true>, grid, dim3(256), 0, s, (const T*)X, (const T*)W, oa, of, M, N, K);
+        bc_launch(gemm_simt_kernel<T, EPI, true>, grid, dim3(256), 0, s, (const T*)X, (const T*)W, oa, of, M, N, K, a, b, cols);
     else
-        bc_launch(gemm_simt_kernel<T, EPI, false>, grid, dim3(256), 0, s, (const T*)X, (const T*)W, oa, of, M, N, K);
+        bc_launch(gemm_simt_kernel<T, EPI, false>, grid, dim3(256), 0, s, (const T*)X, (const T*)W, oa, of, M, N, K, a, b, cols);
     BC_LAUNCH_STATUS();
 }
 
 // X [M, K] and W [N, K] (for SwiGLU: W [2N, K], gate rows then up rows) in the operand
 // type; `out` is [M, N] in the operand type (store, SwiGLU) or float (store_f32, add_f32).
 template <class T>
-static int dispatch(const void* X, const void* W, void* out, int M, int N, int K, int epilogue, cudaStream_t s) {
+static int dispatch(const void* X, const void* W, void* out, int M, int N, int K, int epilogue, float a, float b, int cols, cudaStream_t s) {
     BC_CHECK_ARG(M >= 0 && N > 0 && K > 0, "gemm_simt: bad sizes M=%d N=%d K=%d", M, N, K);
     BC_CHECK_ARG((M + BM - 1) / BM <= 65535, "gemm_simt: %d rows are more than 65535 tiles of %d", M, BM);
     if (M == 0) return BC_OK;
     switch (epilogue) {
-        case EPI_STORE: return launch<T, EPI_STORE>(X, W, out, M, N, K, s);
-        case EPI_STORE_F32: return launch<T, EPI_STORE_F32>(X, W, out, M, N, K, s);
-        case EPI_ADD_F32: return launch<T, EPI_ADD_F32>(X, W, out, M, N, K, s);
-        case EPI_SWIGLU: return launch<T, EPI_SWIGLU>(X, W, out, M, N, K, s);
-        case EPI_RELU2: return launch<T, EPI_RELU2>(X, W, out, M, N, K, s);
+        case EPI_STORE: return launch<T, EPI_STORE>(X, W, out, M, N, K, a, b, cols, s);
+        case EPI_STORE_F32: return launch<T, EPI_STORE_F32>(X, W, out, M, N, K, a, b, cols, s);
+        case EPI_ADD_F32: return launch<T, EPI_ADD_F32>(X, W, out, M, N, K, a, b, cols, s);
+        case EPI_SWIGLU: return launch<T, EPI_SWIGLU>(X, W, out, M, N, K, a, b, cols, s);
+        case EPI_RELU2: return launch<T, EPI_RELU2>(X, W, out, M, N, K, a, b, cols, s);
+        case EPI_XIELU: return launch<T, EPI_XIELU>(X, W, out, M, N, K, a, b, cols, s);
+        case EPI_SILU_F32: return launch<T, EPI_SILU_F32>(X, W, out, M, N, K, a, b, cols, s);
     }
     bc_set_error("gemm_simt: unknown epilogue %d", epilogue);
     return BC_ERR_ARG;
 }
 
 extern "C" int bc_gemm_simt_f32(const void* X, const void* W, void* out, int M, int N, int K, int epilogue, cudaStream_t s) {
-    return dispatch<float>(X, W, out, M, N, K, epilogue, s);
+    BC_CHECK_ARG(epilogue != EPI_XIELU && epilogue != EPI_SILU_F32, "gemm_simt: epilogue %d comes with numbers of its own", epilogue);
+    return dispatch<float>(X, W, out, M, N, K, epilogue, 0.0f, 0.0f, 0, s);
 }
 extern "C" int bc_gemm_simt_bf16(const void* X, const void* W, void* out, int M, int N, int K, int epilogue, cudaStream_t s) {
-    return dispatch<bf16>(X, W, out, M, N, K, epilogue, s);
+    BC_CHECK_ARG(epilogue != EPI_XIELU && epilogue != EPI_SILU_F32, "gemm_simt: epilogue %d comes with numbers of its own", epilogue);
+    return dispatch<bf16>(X, W, out, M, N, K, epilogue, 0.0f, 0.0f, 0, s);
+}
+// The epilogues with numbers of their own: EPI_XIELU (a, b) and EPI_SILU_F32 (cols).
+extern "C" int bc_gemm_simt_act_f32(const void* X, const void* W, void* out, int M, int N, int K, int epilogue, float a, float b, int cols, cudaStream_t s) {
+    return dispatch<float>(X, W, out, M, N, K, epilogue, a, b, cols, s);
+}
+extern "C" int bc_gemm_simt_act_bf16(const void* X, const void* W, void* out, int M, int N, int K, int epilogue, float a, float b, int cols, cudaStream_t s) {
+    return dispatch<bf16>(X, W, out, M, N, K, epilogue, a, b, cols, s);
 }

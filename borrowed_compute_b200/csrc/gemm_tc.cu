@@ -54,6 +54,8 @@ struct TcParams {
     int n_tiles, t_tiles;   // blocks along the weight rows and along the tokens
     int pair_tokens;        // the paired kernel: tokens a tile (64, 128, 192 or 256)
     int starve;             // test hook: the first stage expects 16 bytes that never come, so a bounded wait runs out
+    float act_a, act_b;     // EPI_XIELU: its two numbers
+    int act_cols;           // EPI_SILU_F32: output columns below this one are gated by their own sigmoid
     float glu_limit, glu_alpha;   // SwiGLU: a positive limit bounds gate and up and puts alpha into the gate's sigmoid (see glu_mul)
     long long* trace;       // measurement builds (-DBC_TC_TRACE): sixteen time stamps a block, else null
 };
@@ -276,15 +278,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 if (n >= p.N) return;
                 float r[16];
 #pragma unroll
-                for (int j = 0; j < 16; j++) r[j] = EPI == EPI_SWIGLU ? glu_mul(__uint_as_float(v[j]), __uint_as_float(u[j]), p.glu_limit, p.glu_alpha) : epi_plain<EPI>(__uint_as_float(v[j]));
+                for (int j = 0; j < 16; j++) r[j] = EPI == EPI_SWIGLU ? glu_mul(__uint_as_float(v[j]), __uint_as_float(u[j]), p.glu_limit, p.glu_alpha) : epi_plain<EPI>(__uint_as_float(v[j]), p.act_a, p.act_b, n, p.act_cols);
                 const int t_first = t0 + c0;
                 const size_t o = (size_t)t_first * p.N + n;
 #pragma unroll
                 for (int j = 0; j < 16; j++) {
                     if (t_first + j >= p.T) break;
                     const size_t at = o + (size_t)j * p.N;
-                    if (EPI == EPI_STORE || EPI == EPI_SWIGLU || EPI == EPI_RELU2) ((bf16*)p.out)[at] = __float2bfloat16_rn(r[j]);
-                    if (EPI == EPI_STORE_F32) ((float*)p.out)[at] = r[j];
+                    if (EPI_TO_BF16(EPI)) ((bf16*)p.out)[at] = __float2bfloat16_rn(r[j]);
+                    if (EPI_TO_F32(EPI)) ((float*)p.out)[at] = r[j];
                     // One thread owns each element, so a fire-and-forget reduction gives the same
                     // sum as a load, add and store, without waiting for the load.
                     if (EPI == EPI_ADD_F32) atomicAdd(&((float*)p.out)[at], r[j]);
@@ -350,8 +352,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             auto write = [&](int c, float v, float u) {
                 if (n < p.N) {
                     const size_t o = (size_t)(t0 + c) * p.N + n;
-                    if (EPI == EPI_STORE || EPI == EPI_RELU2) ((bf16*)p.out)[o] = __float2bfloat16_rn(epi_plain<EPI>(v));
-                    if (EPI == EPI_STORE_F32) ((float*)p.out)[o] = v;
+                    if (EPI != EPI_SWIGLU && EPI_TO_BF16(EPI)) ((bf16*)p.out)[o] = __float2bfloat16_rn(epi_plain<EPI>(v, p.act_a, p.act_b, n, p.act_cols));
+                    if (EPI_TO_F32(EPI)) ((float*)p.out)[o] = epi_plain<EPI>(v, p.act_a, p.act_b, n, p.act_cols);
                     if (EPI == EPI_ADD_F32) ((float*)p.out)[o] += v;   // one owner an element: no reduction needed (and measured 0.4 % of a step faster than a fire-and-forget one)
                     if (EPI == EPI_SWIGLU) ((bf16*)p.out)[o] = __float2bfloat16_rn(glu_mul(v, u, p.glu_limit, p.glu_alpha));
                 }
@@ -591,15 +593,15 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 if (out_n >= p.N) return;
                 float r[16];
 #pragma unroll
-                for (int j = 0; j < 16; j++) r[j] = EPI == EPI_SWIGLU ? glu_mul(__uint_as_float(v[j]), __uint_as_float(u[j]), p.glu_limit, p.glu_alpha) : epi_plain<EPI>(__uint_as_float(v[j]));
+                for (int j = 0; j < 16; j++) r[j] = EPI == EPI_SWIGLU ? glu_mul(__uint_as_float(v[j]), __uint_as_float(u[j]), p.glu_limit, p.glu_alpha) : epi_plain<EPI>(__uint_as_float(v[j]), p.act_a, p.act_b, out_n, p.act_cols);
                 const int t_first = t0 + c0;
                 const size_t o = (size_t)t_first * p.N + out_n;
 #pragma unroll
                 for (int j = 0; j < 16; j++) {
                     if (t_first + j >= p.T) break;
                     const size_t at = o + (size_t)j * p.N;
-                    if (EPI == EPI_STORE || EPI == EPI_SWIGLU || EPI == EPI_RELU2) ((bf16*)p.out)[at] = __float2bfloat16_rn(r[j]);
-                    if (EPI == EPI_STORE_F32) ((float*)p.out)[at] = r[j];
+                    if (EPI_TO_BF16(EPI)) ((bf16*)p.out)[at] = __float2bfloat16_rn(r[j]);
+                    if (EPI_TO_F32(EPI)) ((float*)p.out)[at] = r[j];
                     // One thread owns each element, so a fire-and-forget reduction gives the same
                     // sum as a load, add and store, without waiting for the load.
                     if (EPI == EPI_ADD_F32) atomicAdd(&((float*)p.out)[at], r[j]);
@@ -890,11 +892,11 @@ extern "C" void bc_gemm_tc_set_trace(long long* buf, int launches) { g_tc_trace 
 // float by epilogue.  K must be a multiple of 8 (a TMA row stride is a multiple of 16
 // bytes); pointers 16-byte aligned.  splits > 1 needs the workspace above.
 static int gemm_tc_go(const void* X, const void* W, void* out, int T, int N, int K, int epilogue, int splits, float* partial, int* counters,
-                      float glu_limit, float glu_alpha, cudaStream_t s) {
+                      float glu_limit, float glu_alpha, float act_a, float act_b, int act_cols, cudaStream_t s) {
     BC_CHECK_ARG(T >= 0 && N > 0 && K > 0, "gemm_tc: bad sizes T=%d N=%d K=%d", T, N, K);
     BC_CHECK_ARG(K % 8 == 0, "gemm_tc: K=%d is not a multiple of 8 (TMA needs 16-byte row strides); use the CUDA-core product", K);
     BC_CHECK_ARG(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc: operands must be 16-byte aligned");
-    BC_CHECK_ARG(epilogue >= 0 && epilogue <= 4, "gemm_tc: unknown epilogue %d", epilogue);
+    BC_CHECK_ARG(epilogue >= 0 && epilogue <= 6, "gemm_tc: unknown epilogue %d", epilogue);
     BC_CHECK_ARG(splits >= 1, "gemm_tc: bad split count %d", splits);
     if (T == 0) return BC_OK;
     const int bn = bc_gemm_tc_token_tile(T, epilogue);
@@ -923,6 +925,9 @@ static int gemm_tc_go(const void* X, const void* W, void* out, int T, int N, int
     if (!paired) g_tc_starve = 0;
     p.glu_limit = glu_limit;
     p.glu_alpha = glu_alpha;
+    p.act_a = act_a;
+    p.act_b = act_b;
+    p.act_cols = act_cols;
     p.trace = nullptr;
 #ifdef BC_TC_TRACE
     if (!paired && g_tc_trace && g_tc_trace_next < g_tc_trace_launches) p.trace = g_tc_trace + (size_t)(g_tc_trace_next++) * 1024 * 16;
@@ -934,6 +939,8 @@ static int gemm_tc_go(const void* X, const void* W, void* out, int T, int N, int
             case EPI_ADD_F32: return launch_pair<EPI_ADD_F32>(mw, mx, p, s);
             case EPI_SWIGLU: return launch_pair<EPI_SWIGLU>(mw, mx, p, s);
             case EPI_RELU2: return launch_pair<EPI_RELU2>(mw, mx, p, s);
+            case EPI_XIELU: return launch_pair<EPI_XIELU>(mw, mx, p, s);
+            case EPI_SILU_F32: return launch_pair<EPI_SILU_F32>(mw, mx, p, s);
         }
     }
     switch (epilogue) {
@@ -942,19 +949,28 @@ static int gemm_tc_go(const void* X, const void* W, void* out, int T, int N, int
         case EPI_ADD_F32: return launch_bn<EPI_ADD_F32>(bn, stack, mw, mx, p, splits, s);
         case EPI_SWIGLU: return launch_bn<EPI_SWIGLU>(bn, false, mw, mx, p, splits, s);
         case EPI_RELU2: return launch_bn<EPI_RELU2>(bn, stack, mw, mx, p, splits, s);
+        case EPI_XIELU: return launch_bn<EPI_XIELU>(bn, stack, mw, mx, p, splits, s);
+        case EPI_SILU_F32: return launch_bn<EPI_SILU_F32>(bn, stack, mw, mx, p, splits, s);
     }
     return BC_ERR_ARG;
 }
 
 extern "C" int bc_gemm_tc_bf16(const void* X, const void* W, void* out, int T, int N, int K, int epilogue, int splits, float* partial,
                                int* counters, cudaStream_t s) {
-    return gemm_tc_go(X, W, out, T, N, K, epilogue, splits, partial, counters, 0.0f, 1.0f, s);
+    BC_CHECK_ARG(epilogue != EPI_XIELU && epilogue != EPI_SILU_F32, "gemm_tc: epilogue %d comes with numbers of its own", epilogue);
+    return gemm_tc_go(X, W, out, T, N, K, epilogue, splits, partial, counters, 0.0f, 1.0f, 0.0f, 0.0f, 0, s);
 }
 // The gated product (EPI_SWIGLU) with bounds: out = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit).
 extern "C" int bc_gemm_tc_glu_bf16(const void* X, const void* W, void* out, int T, int N, int K, int splits, float* partial, int* counters,
                                    float limit, float alpha, cudaStream_t s) {
     BC_CHECK_ARG(limit > 0.0f, "gemm_tc: the bound of a gated product must be positive, got %g", (double)limit);
-    return gemm_tc_go(X, W, out, T, N, K, EPI_SWIGLU, splits, partial, counters, limit, alpha, s);
+    return gemm_tc_go(X, W, out, T, N, K, EPI_SWIGLU, splits, partial, counters, limit, alpha, 0.0f, 0.0f, 0, s);
+}
+// The epilogues with numbers of their own: EPI_XIELU (a, b) and EPI_SILU_F32 (cols).
+extern "C" int bc_gemm_tc_act_bf16(const void* X, const void* W, void* out, int T, int N, int K, int epilogue, int splits, float* partial, int* counters,
+                                   float a, float b, int cols, cudaStream_t s) {
+    BC_CHECK_ARG(epilogue == EPI_XIELU || epilogue == EPI_SILU_F32, "gemm_tc: epilogue %d has no numbers", epilogue);
+    return gemm_tc_go(X, W, out, T, N, K, epilogue, splits, partial, counters, 0.0f, 1.0f, a, b, cols, s);
 }
 
 // ------------------------------------------------------------ the product over groups of rows

@@ -3,10 +3,11 @@
 //     S_t = diag(a_t) S_(t-1) + (c_t k_t) v_t^T        o_t = f S_t^T q_t + d v_t
 //
 // per head, with S [N, P] (N key channels, P value channels) in float, carried from token to token for every
-// sequence.  Two designs are this recurrence:
+// sequence.  Three designs are this recurrence:
 //   - gated linear attention: a_t a vector of N decays, c = 1, d = 0, f = N^(-1/2), q, k, v per head;
 //   - the state-space dual form (Mamba-2): a_t = exp(-exp(A_log) dt_t) one number a head, c_t = dt_t, k = B and
-//     q = C shared by the heads of a group, v = x, d = D of the head.
+//     q = C shared by the heads of a group, v = x, d = D of the head;
+//   - lightning attention: a_t one constant a head (one row of decays that every token reads: stride 0), c = f = 1, d = 0.
 // Everything here is float: decays, step sizes, the state and all sums.
 //
 // Kernels:
@@ -14,8 +15,8 @@
 //   ssd_prepare    causal convolution with bias and silu over [x | B | C], its last inputs kept per sequence;
 //                  dt = softplus(. + dt_bias) and the decay exp(-exp(A_log) dt)
 //   gla_decay      sigmoid(z)^(1/tau), z = W_2 inner + b, as exp(-softplus(-z) / tau)
-//   gated_norm     a row in equal parts, each over its root mean square, times a weight, the gate silu(g) before
-//                  or after the norm, a factor on the result; float in, activation type out
+//   gated_norm     a row in equal parts, each over its root mean square, times a weight, the gate silu(g) or sigmoid(g)
+//                  before or after the norm, a factor on the result; float in, activation type out
 #include "common.cuh"
 
 #define SCAN_NT 8          // threads that share a value channel, each with every eighth key channel
@@ -331,12 +332,12 @@ ssd_prepare_kernel(const float* __restrict__ proj, int stride, int conv_at, int 
     }
 }
 
-// weight_t: [taps, C] (tap by tap; the last is the current token's); bias: [C] or null; dt_bias, a_log: [H];
+// weight_t: [taps, C] (tap by tap; the last is the current token's); bias: [C] or null; dt_bias, a_log: [H] (H = 0: no step sizes);
 // tail: [slots, taps - 1, C]; xbc: [rows, C]; dtda: [rows, 2 H].
 extern "C" int bc_ssd_prepare(const float* proj, int stride, int conv_at, int dt_at, const float* weight_t, const float* bias, const float* dt_bias,
                               const float* a_log, float* tail, const int* seq_rows, const int* seq_slot, float* xbc, float* dtda, int seqs,
                               int max_new, int C, int H, int taps, int n_slots, int write_tail, cudaStream_t s) {
-    BC_CHECK_ARG(seqs >= 0 && seqs <= 65535 && max_new >= 0 && C > 0 && H > 0, "ssd_prepare: bad sizes seqs=%d max_new=%d C=%d H=%d", seqs, max_new, C, H);
+    BC_CHECK_ARG(seqs >= 0 && seqs <= 65535 && max_new >= 0 && C > 0 && H >= 0, "ssd_prepare: bad sizes seqs=%d max_new=%d C=%d H=%d", seqs, max_new, C, H);
     BC_CHECK_ARG(taps >= 1 && taps <= SSD_MAX_TAPS, "ssd_prepare: %d taps are outside 1 to %d", taps, SSD_MAX_TAPS);
     if (seqs == 0 || max_new == 0) return BC_OK;
     const int tiles = (max_new + SSD_TILE - 1) / SSD_TILE;
@@ -383,11 +384,13 @@ extern "C" int bc_gla_decay(const float* proj, int stride, int inner_at, const f
 // -------------------------------------------------------------------------------- gated_norm
 // y: [rows, W] float; gate: row r's at gate + r * g_stride; weight: `period` values, repeated over the row (period = W: one
 // a column; period = W / parts: shared by the parts); row_slot (may be null): rows whose slot is negative give zeros.  Block (part, row): z = y (* silu(g) if gate_first); z over the root mean
-// square of the part, eps inside the root; times weight (times silu(g) if not gate_first); times factor.
+// square of the part, eps inside the root; times weight (times silu(g) if not gate_first); times factor.  With plain_sigmoid the
+// gate is sigmoid(g).
 template <class T>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, int g_stride, const float* __restrict__ weight, int period,
-                  const int* __restrict__ row_slot, T* __restrict__ out, int W, int part, float eps, int gate_first, float factor) {
+                  const int* __restrict__ row_slot, T* __restrict__ out, int W, int part, float eps, int gate_first, int plain_sigmoid,
+                  float factor) {
     __shared__ float scratch[32];
     pdl_launch_dependents_if_resident();
     pdl_wait();
@@ -405,14 +408,14 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
         float z = yr[c];
         if (gate_first) {
             const float g = gr[c];
-            z *= g / (1.0f + expf(-g));
+            z *= (plain_sigmoid ? 1.0f : g) / (1.0f + expf(-g));
         }
         ss = fmaf(z, z, ss);
     }
     const float scale = factor / sqrtf(block_sum(ss, scratch) / (float)part + eps);
     for (int c = threadIdx.x; c < part; c += blockDim.x) {
         const float g = gr[c];
-        const float sg = g / (1.0f + expf(-g));
+        const float sg = (plain_sigmoid ? 1.0f : g) / (1.0f + expf(-g));
         const float z = gate_first ? yr[c] * sg : yr[c];
         const float o = z * scale * weight[(c0 + c) % period];
         out[(size_t)r * W + c0 + c] = from_f32<T>(gate_first ? o : o * sg);
@@ -421,7 +424,7 @@ gated_norm_kernel(const float* __restrict__ y, const float* __restrict__ gate, i
 
 template <class T>
 static int gated_norm(const float* y, const float* gate, int g_stride, const float* weight, int period, const int* row_slot, void* out, int rows,
-                      int W, int parts, float eps, int gate_first, float factor, cudaStream_t s) {
+                      int W, int parts, float eps, int gate_first, int plain_sigmoid, float factor, cudaStream_t s) {
     BC_CHECK_ARG(rows >= 0 && rows <= 2147483647 && W > 0 && parts > 0 && parts <= 65535 && W % parts == 0, "gated_norm: bad sizes rows=%d W=%d parts=%d", rows, W, parts);
     BC_CHECK_ARG(period > 0 && (period == W || period == W / parts), "gated_norm: a weight of %d values fits neither the row nor a part", period);
     if (rows == 0) return BC_OK;
@@ -431,15 +434,15 @@ static int gated_norm(const float* y, const float* gate, int g_stride, const flo
     for (int at = 0; at < rows; at += 65535) {
         const int n = rows - at < 65535 ? rows - at : 65535;
         bc_launch(gated_norm_kernel<T>, dim3(parts, n), dim3(threads), 0, s, y + (size_t)at * W, gate + (size_t)at * g_stride, g_stride, weight, period,
-                  row_slot ? row_slot + at : nullptr, (T*)out + (size_t)at * W, W, part, eps, gate_first, factor);
+                  row_slot ? row_slot + at : nullptr, (T*)out + (size_t)at * W, W, part, eps, gate_first, plain_sigmoid, factor);
     }
     BC_LAUNCH_STATUS();
 }
 extern "C" int bc_gated_norm_f32(const float* y, const float* gate, int g_stride, const float* weight, int period, const int* row_slot, void* out,
-                                 int rows, int W, int parts, float eps, int gate_first, float factor, cudaStream_t s) {
-    return gated_norm<float>(y, gate, g_stride, weight, period, row_slot, out, rows, W, parts, eps, gate_first, factor, s);
+                                 int rows, int W, int parts, float eps, int gate_first, int plain_sigmoid, float factor, cudaStream_t s) {
+    return gated_norm<float>(y, gate, g_stride, weight, period, row_slot, out, rows, W, parts, eps, gate_first, plain_sigmoid, factor, s);
 }
 extern "C" int bc_gated_norm_bf16(const float* y, const float* gate, int g_stride, const float* weight, int period, const int* row_slot, void* out,
-                                  int rows, int W, int parts, float eps, int gate_first, float factor, cudaStream_t s) {
-    return gated_norm<bf16>(y, gate, g_stride, weight, period, row_slot, out, rows, W, parts, eps, gate_first, factor, s);
+                                  int rows, int W, int parts, float eps, int gate_first, int plain_sigmoid, float factor, cudaStream_t s) {
+    return gated_norm<bf16>(y, gate, g_stride, weight, period, row_slot, out, rows, W, parts, eps, gate_first, plain_sigmoid, factor, s);
 }

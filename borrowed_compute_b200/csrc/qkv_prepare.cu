@@ -189,19 +189,20 @@ extern "C" int bc_qkv_prepare_bf16(const float* qkv, const float* bias, const fl
 // the rotation of the first `rot` dimensions, then q to the activation type and k, v into the cache.
 // `pairing` 0 pairs dimension i with i + rot/2, 1 pairs 2i with 2i + 1.  One warp a (row, head): the lanes
 // take pairs of dimensions, so the sum of squares and the rotation need no second pass over memory; which
-// values a lane adds, and in which order, depends on the sizes alone.
+// values a lane adds, and in which order, depends on the sizes alone.  Values may have a number of heads of their own (VG: two
+// key maps that share one value head, say), and a layer that reads another layer's cache projects queries alone (G = VG = 0).
 template <class T>
 __global__ void __launch_bounds__(256)
 qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                          const float* __restrict__ cos_sin, int n_positions, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                          const int* __restrict__ page_table, int max_pages, int n_pages, T* __restrict__ q_out, T* __restrict__ k_cache,
-                         T* __restrict__ v_cache, int H, int G, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache) {
+                         T* __restrict__ v_cache, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache) {
     pdl_launch_dependents_if_resident();
     pdl_wait();
     PDL_FRESH(qkv);
     const int r = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const int nq = H * D, nk = G * D, nv = G * DV;
+    const int nq = H * D, nk = G * D, nv = VG * DV;
     const float* x = qkv + (size_t)r * (nq + nk + nv);
     const int slot = row_slot[r];
     const int pos = row_pos[r];
@@ -247,7 +248,7 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
     if (cache) {
         for (int i = threadIdx.x; i < nv; i += blockDim.x) {
             const int g = i / DV, d = i - g * DV;
-            v_cache[(((size_t)page * G + g) * BC_PAGE + pos % BC_PAGE) * DV + d] = from_f32<T>(x[nq + nk + i]);
+            v_cache[(((size_t)page * VG + g) * BC_PAGE + pos % BC_PAGE) * DV + d] = from_f32<T>(x[nq + nk + i]);
         }
     }
 }
@@ -255,30 +256,31 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
 template <class T>
 static int launch_heads(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_sin, int n_positions, const int* row_pos,
                         const int* row_slot, const int* page_table, int max_pages, int n_pages, void* q_out, void* k_cache, void* v_cache, int rows,
-                        int H, int G, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache, cudaStream_t s) {
-    BC_CHECK_ARG(rows >= 0 && H > 0 && G > 0 && D > 0 && DV > 0, "qkv_prepare_heads: bad sizes rows=%d H=%d G=%d D=%d DV=%d", rows, H, G, D, DV);
+                        int H, int G, int VG, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache, cudaStream_t s) {
+    BC_CHECK_ARG(rows >= 0 && H > 0 && G >= 0 && VG >= 0 && (G > 0) == (VG > 0) && D > 0 && DV > 0, "qkv_prepare_heads: bad sizes rows=%d H=%d G=%d D=%d DV=%d", rows, H, G, D, DV);
     BC_CHECK_ARG(rot >= 0 && rot % 2 == 0 && rot <= D, "qkv_prepare_heads: %d rotated dimensions of a head of %d", rot, D);
-    BC_CHECK_ARG(!normed || (q_weight && k_weight), "qkv_prepare_heads: the norm needs its weights");
+    BC_CHECK_ARG(!normed || (q_weight && (k_weight || G == 0)), "qkv_prepare_heads: the norm needs its weights");
     if (rows == 0) return BC_OK;
     const int heads = H + G;
     const int threads = heads >= 8 ? 256 : heads >= 4 ? 128 : 64;      // by the row's heads alone
     bc_launch(qkv_prepare_heads_kernel<T>, dim3(rows), dim3(threads), 0, s, qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot,
-              page_table, max_pages, n_pages, (T*)q_out, (T*)k_cache, (T*)v_cache, H, G, D, DV, rot, pairing, eps, normed, write_cache);
+              page_table, max_pages, n_pages, (T*)q_out, (T*)k_cache, (T*)v_cache, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache);
     BC_LAUNCH_STATUS();
 }
 
-// As bc_qkv_prepare_*, without biases; q_weight and k_weight hold D values each; cos_sin: [n_positions, rot / 2, 2].
+// As bc_qkv_prepare_*, without biases; q_weight and k_weight hold D values each; cos_sin: [n_positions, rot / 2, 2];
+// qkv: [rows, H D + G D + VG DV]; v_cache: [pages, VG, PAGE, DV].
 extern "C" int bc_qkv_prepare_heads_f32(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_sin, int n_positions,
                                         const int* row_pos, const int* row_slot, const int* page_table, int max_pages, int n_pages, void* q_out,
-                                        void* k_cache, void* v_cache, int rows, int H, int G, int D, int DV, int rot, int pairing, float eps,
+                                        void* k_cache, void* v_cache, int rows, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps,
                                         int normed, int write_cache, cudaStream_t s) {
     return launch_heads<float>(qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot, page_table, max_pages, n_pages, q_out, k_cache,
-                               v_cache, rows, H, G, D, DV, rot, pairing, eps, normed, write_cache, s);
+                               v_cache, rows, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, s);
 }
 extern "C" int bc_qkv_prepare_heads_bf16(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_sin, int n_positions,
                                          const int* row_pos, const int* row_slot, const int* page_table, int max_pages, int n_pages, void* q_out,
-                                         void* k_cache, void* v_cache, int rows, int H, int G, int D, int DV, int rot, int pairing, float eps,
+                                         void* k_cache, void* v_cache, int rows, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps,
                                          int normed, int write_cache, cudaStream_t s) {
     return launch_heads<bf16>(qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot, page_table, max_pages, n_pages, q_out, k_cache,
-                              v_cache, rows, H, G, D, DV, rot, pairing, eps, normed, write_cache, s);
+                              v_cache, rows, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, s);
 }

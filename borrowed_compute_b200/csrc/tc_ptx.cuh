@@ -7,10 +7,16 @@
 
 #include "common.cuh"
 
-enum { EPI_STORE = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_RELU2 = 4 };
+enum { EPI_STORE = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_RELU2 = 4, EPI_XIELU = 5, EPI_SILU_F32 = 6 };
+// Which epilogues store the activation type, and which store floats.
+#define EPI_TO_BF16(E) ((E) == EPI_STORE || (E) == EPI_SWIGLU || (E) == EPI_RELU2 || (E) == EPI_XIELU)
+#define EPI_TO_F32(E) ((E) == EPI_STORE_F32 || (E) == EPI_SILU_F32)
 // What an epilogue without a second operand does to a full sum before it is stored: EPI_RELU2 squares what is above zero (in
-// float; the store rounds once), the others leave it.
-template <int EPI> __device__ __forceinline__ float epi_plain(float v) {
+// float; the store rounds once); EPI_XIELU is a v^2 + v/2 above zero and b (e^v - 1 - v) + v/2 below; EPI_SILU_F32 gates output columns
+// n < cols by their own sigmoid and stores floats; the others leave it.
+template <int EPI> __device__ __forceinline__ float epi_plain(float v, float a = 0.0f, float b = 0.0f, int n = 0, int cols = 0) {
+    if (EPI == EPI_XIELU) return fmaf(0.5f, v, v > 0.0f ? a * v * v : b * (__expf(v) - 1.0f - v));
+    if (EPI == EPI_SILU_F32) return n < cols ? __fdividef(v, 1.0f + __expf(-v)) : v;
     if (EPI == EPI_RELU2) {
         v = fmaxf(v, 0.0f);
         return v * v;

@@ -10,6 +10,7 @@ import torch
 
 from ..architectures import resolve
 from ..parts import base as P
+from ..parts.streams import StreamBundle
 from ..parts.base import (BLOCKS, EMBEDDINGS, HEADS, JUNCTIONS, NORMS, POSITION_ENCODINGS, CacheNeed, ModelSpec, PartSpec, Runtime, StateNeed,
                           StepContext, TensorSpec)
 
@@ -27,8 +28,14 @@ class DecoderModel:
             if run.memory_of is not None and not (0 <= run.memory_of < i and spec.schedule[run.memory_of].memory_of is None):
                 raise ValueError(f"schedule entry {i} reads the memory of entry {run.memory_of}, which is not an earlier owner")
         self.embedding = _build(EMBEDDINGS, spec.embedding)
+        self.embedding_norm = None if spec.embedding_norm is None else _build(NORMS, spec.embedding_norm)
         self.position = None if spec.position is None else _build(POSITION_ENCODINGS, spec.position)
         self.blocks = [BLOCKS.get(layer.block).build(layer, spec.hidden_size) for layer in spec.layers]
+        for layer, block in zip(spec.layers, self.blocks):
+            if block.STREAMS != (spec.streams > 0):
+                raise ValueError(f"block '{layer.block}' runs on {'a bundle of streams' if block.STREAMS else 'one residual stream'}, the model has {spec.streams or 'one plain stream'}")
+        if spec.streams and (spec.junctions or spec.position is not None):
+            raise ValueError("a bundle of streams takes no junctions and no position encoding on the embeddings")
         self.junctions = [_build(JUNCTIONS, j) for j in spec.junctions]
         for i, run in enumerate(spec.schedule):
             if run.enter is not None and not 0 <= run.enter[0] < len(self.junctions):
@@ -37,12 +44,14 @@ class DecoderModel:
         self.head = _build(HEADS, spec.head)
         self.rt: Optional[Runtime] = None
         # For looking inside a step: called as after_run(schedule entry, residual) when a run has added to the stream
-        # (an eager step only; a captured step replays without it).
+        # (an eager step only; a captured step replays without it); where the stream is a bundle, residual is the sum of its copies.
         self.after_run = None
 
     def named_parts(self):
         """(tensor-name prefix, part) of every part of the model; each block lists its own."""
         yield self.spec.embedding.prefix, self.embedding
+        if self.embedding_norm is not None:
+            yield self.spec.embedding_norm.prefix, self.embedding_norm
         if self.position is not None:
             yield self.spec.position.prefix, self.position
         for layer, block in zip(self.spec.layers, self.blocks):
@@ -74,6 +83,10 @@ class DecoderModel:
             needs.append(None if mixer is None else mixer.cache_need())
             states.append(None if mixer is None else mixer.state_need())
             memory_of.append(run.memory_of)
+        # A run that reads another's memory may see further back than its owner: the owner keeps what both read.
+        for i, j in enumerate(memory_of):
+            if j is not None and needs[j] is not None and needs[i] is not None:
+                needs[j] = needs[j].widened(needs[i])
         return needs, states, memory_of
 
     def more_state_needs(self) -> List[Dict[str, StateNeed]]:
@@ -85,6 +98,10 @@ class DecoderModel:
         rt = self.rt
         residual = torch.empty((ctx.rows, self.spec.hidden_size), dtype=torch.float32, device=rt.device)
         self.embedding.forward(ctx, residual)
+        if self.spec.streams:
+            return self._forward_streams(residual, ctx, cache, want_rows, n_want)
+        if self.embedding_norm is not None:
+            self.embedding_norm.forward(residual.clone(), residual)
         if self.position is not None:
             self.position.on_embeddings(residual, ctx)
         embedded = None
@@ -100,9 +117,25 @@ class DecoderModel:
                 self.after_run(i, residual)
         h = torch.empty((n_want, self.spec.hidden_size), dtype=rt.dtype, device=rt.device)
         self.final_norm.forward(residual, h, want_rows)
-        scores = torch.empty((n_want, self.spec.vocab_size), dtype=torch.float32, device=rt.device)
+        return self._scores(h)
+
+    def _scores(self, h: torch.Tensor) -> torch.Tensor:
+        scores = torch.empty((h.shape[0], self.spec.vocab_size), dtype=torch.float32, device=self.rt.device)
         self.head.forward(h, scores, self.embedding.table())
         return scores
+
+    def _forward_streams(self, embedded: torch.Tensor, ctx: StepContext, cache, want_rows: Optional[torch.Tensor], n_want: int) -> torch.Tensor:
+        """``forward`` where a row's residual stream is a bundle of copies."""
+        rt = self.rt
+        bundle = StreamBundle(ctx.rows, self.spec.streams, self.spec.hidden_size, rt.device)
+        bundle.start(embedded, self.embedding_norm)
+        for i, run in enumerate(self.spec.schedule):
+            self.blocks[run.layer].forward(bundle, ctx, cache.memory(i), rt)
+            if self.after_run is not None and not ctx.extras.get("graph"):
+                self.after_run(i, bundle.total())
+        h = torch.empty((n_want, self.spec.hidden_size), dtype=rt.dtype, device=rt.device)
+        bundle.finish(self.final_norm, h, want_rows)
+        return self._scores(h)
 
 
 def model_for_config(config: Mapping[str, Any], shapes: Optional[Mapping[str, tuple]] = None) -> Tuple[Any, DecoderModel]:

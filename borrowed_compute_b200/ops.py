@@ -17,7 +17,8 @@ from .csrc import build as _build
 
 PAGE = 64  # tokens per cache page; checked against the library at load
 
-EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_RELU2 = 0, 1, 2, 3, 4
+EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_RELU2, EPI_XIELU, EPI_SILU_F32 = 0, 1, 2, 3, 4, 5, 6
+_EPI_FLOAT = (EPI_STORE_F32, EPI_ADD_F32, EPI_SILU_F32)      # epilogues whose output is float32 whatever the operands are
 
 _c_int, _c_float, _c_void_p = ctypes.c_int, ctypes.c_float, ctypes.c_void_p
 
@@ -151,7 +152,8 @@ label = ""
 _CLASS_OF = {
     "bc_embed": "embedding", "bc_rmsnorm": "norm", "bc_swiglu": "activation", "bc_rope_append": "rotary + append",
     "bc_attention_rows": "attention", "bc_attention_decode": "attention", "bc_attention_prefill": "attention",
-    "bc_short_conv": "short convolution", "bc_norm_pair": "norm", "bc_delta": "delta rule", "bc_polynorm": "activation", "bc_qkv_prepare": "rotary + append",
+    "bc_short_conv": "short convolution", "bc_norm_pair": "norm", "bc_delta_split": "low-rank split", "bc_delta": "delta rule",
+    "bc_hyper": "streams + norm", "bc_diff": "attention", "bc_polynorm": "activation", "bc_qkv_prepare": "rotary + append",
     "bc_linear_scan": "recurrence", "bc_ssd_prepare": "recurrence set-up", "bc_gla_decay": "recurrence set-up", "bc_gated_norm": "gated norm",
     "bc_moe_product": "expert product", "bc_gemm_tc_grouped": "expert product", "bc_moe_route": "routing", "bc_moe_plan": "expert sort",
     "bc_moe_gather": "expert gather", "bc_moe_combine": "expert sum", "bc_softcap": "softcap", "bc_reentry": "re-entry",
@@ -280,11 +282,23 @@ def random_normal(out: torch.Tensor, key: int, std: float) -> None:
 
 # ---------------------------------------------------------------------------------- products
 
-def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int) -> None:
+def _act_numbers(who: str, epilogue: int, act: Optional[Tuple[float, float]], cols: Optional[int]) -> Optional[Tuple[float, float, int]]:
+    """(a, b, cols) for the epilogues that have numbers of their own, None for the others."""
+    if (epilogue == EPI_XIELU) != (act is not None) or (epilogue == EPI_SILU_F32) != (cols is not None):
+        raise KernelError(f"{who}: EPI_XIELU comes with act=(a, b), EPI_SILU_F32 with cols, no other epilogue with either")
+    if act is None and cols is None:
+        return None
+    return (0.0, 0.0, int(cols)) if act is None else (float(act[0]), float(act[1]), 0)
+
+
+def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, act: Optional[Tuple[float, float]] = None,
+              cols: Optional[int] = None) -> None:
     """out = x @ w.T on the CUDA cores with float accumulation in ascending k.
     EPI_STORE: out in x's type; EPI_STORE_F32: float32; EPI_ADD_F32: out += (float32);
     EPI_SWIGLU: w stacks gate rows on up rows, out[:, j] = silu(g_j) * u_j in x's type;
-    EPI_RELU2: out = max(sum, 0)^2 in x's type, squared in float and rounded once."""
+    EPI_RELU2: out = max(sum, 0)^2 in x's type, squared in float and rounded once;
+    EPI_XIELU (``act`` = (a, b)): out = a s^2 + s/2 for sums s above zero, b (e^s - 1 - s) + s/2 below, in x's type;
+    EPI_SILU_F32 (``cols``): float32, columns below ``cols`` times their own sigmoid."""
     _need(x, "x")
     _need(w, "w", x.dtype)
     M, K = x.shape
@@ -292,9 +306,15 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int
     N = n_w // 2 if epilogue == EPI_SWIGLU else n_w
     if w.shape[1] != K or (epilogue == EPI_SWIGLU and n_w % 2):
         raise KernelError(f"gemm: x is {tuple(x.shape)}, w is {tuple(w.shape)}")
-    _need(out, "out", torch.float32 if epilogue in (EPI_STORE_F32, EPI_ADD_F32) else x.dtype)
+    _need(out, "out", torch.float32 if epilogue in _EPI_FLOAT else x.dtype)
     if tuple(out.shape) != (M, N):
         raise KernelError(f"gemm: out is {tuple(out.shape)}, wanted {(M, N)}")
+    numbers = _act_numbers("gemm_simt", epilogue, act, cols)
+    if numbers is not None:
+        a, b, n_cols = numbers
+        _call(_fn("bc_gemm_simt_act_" + _suffix(x.dtype)), _ptr(x), _ptr(w), _ptr(out), _c_int(M), _c_int(N), _c_int(K), _c_int(epilogue), _c_float(a),
+              _c_float(b), _c_int(n_cols), _stream())
+        return
     _call(_fn("bc_gemm_simt_" + _suffix(x.dtype)), _ptr(x), _ptr(w), _ptr(out), _c_int(M), _c_int(N), _c_int(K), _c_int(epilogue), _stream())
 
 
@@ -365,7 +385,7 @@ def gemm_tc_splits(T: int, N: int, K: int, epilogue: int) -> int:
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, splits: Optional[int] = None,
-            glu: Optional[Tuple[float, float]] = None) -> None:
+            glu: Optional[Tuple[float, float]] = None, act: Optional[Tuple[float, float]] = None, cols: Optional[int] = None) -> None:
     """out = x @ w.T for bf16 operands on the tcgen05 tensor cores (float accumulation in
     TMEM), with the epilogues of gemm_simt.  ``splits`` > 1 cuts K across blocks that add
     their partial sums in a fixed order.  ``glu`` = (limit, alpha) turns EPI_SWIGLU's gate into the bounded one:
@@ -377,7 +397,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
     N = n_w // 2 if epilogue == EPI_SWIGLU else n_w
     if w.shape[1] != K or (epilogue == EPI_SWIGLU and n_w % 2):
         raise KernelError(f"gemm: x is {tuple(x.shape)}, w is {tuple(w.shape)}")
-    _need(out, "out", torch.float32 if epilogue in (EPI_STORE_F32, EPI_ADD_F32) else torch.bfloat16)
+    _need(out, "out", torch.float32 if epilogue in _EPI_FLOAT else torch.bfloat16)
     if tuple(out.shape) != (M, N):
         raise KernelError(f"gemm: out is {tuple(out.shape)}, wanted {(M, N)}")
     if M == 0:
@@ -397,6 +417,12 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, 
             raise KernelError("gemm_tc: bounds come with the gated product (EPI_SWIGLU)")
         _call(_fn("bc_gemm_tc_glu_bf16"), _ptr(x), _ptr(w), _ptr(out), _c_int(M), _c_int(N), _c_int(K), _c_int(splits), _ptr(partial), _ptr(counters),
               _c_float(glu[0]), _c_float(glu[1]), _stream())
+        return
+    numbers = _act_numbers("gemm_tc", epilogue, act, cols)
+    if numbers is not None:
+        a, b, n_cols = numbers
+        _call(_fn("bc_gemm_tc_act_bf16"), _ptr(x), _ptr(w), _ptr(out), _c_int(M), _c_int(N), _c_int(K), _c_int(epilogue), _c_int(splits), _ptr(partial),
+              _ptr(counters), _c_float(a), _c_float(b), _c_int(n_cols), _stream())
         return
     _call(_fn("bc_gemm_tc_bf16"), _ptr(x), _ptr(w), _ptr(out), _c_int(M), _c_int(N), _c_int(K), _c_int(epilogue), _c_int(splits),
           _ptr(partial), _ptr(counters), _stream())
@@ -508,8 +534,15 @@ def self_check(device: torch.device) -> None:
             product(xb, wb, gated, EPI_SWIGLU)
             squared = torch.empty((n, 2 * rows_w), dtype=torch.bfloat16, device=device)
             product(xb, wb, squared, EPI_RELU2)
+            curved = torch.empty((n, 2 * rows_w), dtype=torch.bfloat16, device=device)
+            product(xb, wb, curved, EPI_XIELU, act=(0.75, 1.25))
+            curve = np.where(full > 0, 0.75 * full * full, 1.25 * (np.expm1(np.minimum(full, 0.0)) - np.minimum(full, 0.0))) + 0.5 * full
+            gated_cols = torch.empty((n, 2 * rows_w), dtype=torch.float32, device=device)
+            product(xb, wb, gated_cols, EPI_SILU_F32, cols=41)
+            partly = np.where(np.arange(2 * rows_w) < 41, full / (1.0 + np.exp(-full)), full)
             checks = {"store": bad(stored, full, rounded), "store_f32": bad(scores, full), "add_f32": bad(added, full + 0.25),
-                      "swiglu": bad(gated, gate / (1.0 + np.exp(-gate)) * up, rounded), "relu2": bad(squared, np.maximum(full, 0.0) ** 2, rounded)}
+                      "swiglu": bad(gated, gate / (1.0 + np.exp(-gate)) * up, rounded), "relu2": bad(squared, np.maximum(full, 0.0) ** 2, rounded),
+                      "xielu": bad(curved, curve, rounded), "silu_f32": bad(gated_cols, partly)}
             wrong = [k for k, v in checks.items() if v]
             if wrong:
                 raise KernelError(f"self-check: the {name} product with {n} row(s) is wrong for the epilogue(s) {wrong} on a "
@@ -757,28 +790,33 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
 
 
 def qkv_prepare_heads(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], cos_sin: Optional[torch.Tensor],
-                      row_pos: torch.Tensor, row_slot: torch.Tensor, page_table: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor,
-                      v_cache: torch.Tensor, heads: int, kv_heads: int, head_dim: int, value_dim: int, rot_dims: int, pairing: int, eps: float,
-                      write_cache: bool = True) -> None:
+                      row_pos: torch.Tensor, row_slot: torch.Tensor, page_table: torch.Tensor, q_out: torch.Tensor, k_cache: Optional[torch.Tensor],
+                      v_cache: Optional[torch.Tensor], heads: int, kv_heads: int, head_dim: int, value_dim: int, rot_dims: int, pairing: int, eps: float,
+                      write_cache: bool = True, value_heads: Optional[int] = None) -> None:
     """Between the fused projection (float32) and attention for models that normalise every head by itself: an RMS norm of each
     head of q and of k over its ``head_dim`` values with weights of that many values shared by the heads (when given), rotation of
     the first ``rot_dims`` dimensions of each head (``pairing`` 0: i with i + rot_dims/2; 1: 2i with 2i + 1), q into ``q_out`` and
-    k, v into the rows' places in the paged cache."""
+    k, v into the rows' places in the paged cache.  ``value_heads`` (default: ``kv_heads``) heads of values follow the keys;
+    ``kv_heads`` 0: the projection holds queries alone and nothing is cached."""
+    value_heads = kv_heads if value_heads is None else int(value_heads)
     _need(qkv, "qkv", torch.float32)
     _need(q_out, "q_out")
-    _need(k_cache, "k_cache", q_out.dtype)
-    _need(v_cache, "v_cache", q_out.dtype)
     _need(row_pos, "row_pos", torch.int32)
     _need(row_slot, "row_slot", torch.int32)
     _need(page_table, "page_table", torch.int32)
     rows = qkv.shape[0]
-    nq, nk, nv = heads * head_dim, kv_heads * head_dim, kv_heads * value_dim
+    nq, nk, nv = heads * head_dim, kv_heads * head_dim, value_heads * value_dim
     if qkv.shape[1] != nq + nk + nv or tuple(q_out.shape) != (rows, nq):
         raise KernelError(f"qkv_prepare_heads: qkv {tuple(qkv.shape)} or q_out {tuple(q_out.shape)} do not fit the head sizes")
-    if tuple(k_cache.shape[1:]) != (kv_heads, PAGE, head_dim) or tuple(v_cache.shape) != (k_cache.shape[0], kv_heads, PAGE, value_dim):
-        raise KernelError(f"qkv_prepare_heads: cache is {tuple(k_cache.shape)} and {tuple(v_cache.shape)}")
-    if (q_weight is None) != (k_weight is None):
-        raise KernelError("qkv_prepare_heads: the norm needs both weights or none")
+    n_pages = 0
+    if kv_heads > 0:
+        _need(k_cache, "k_cache", q_out.dtype)
+        _need(v_cache, "v_cache", q_out.dtype)
+        n_pages = k_cache.shape[0]
+        if tuple(k_cache.shape[1:]) != (kv_heads, PAGE, head_dim) or tuple(v_cache.shape) != (n_pages, value_heads, PAGE, value_dim):
+            raise KernelError(f"qkv_prepare_heads: cache is {tuple(k_cache.shape)} and {tuple(v_cache.shape)}")
+        if (q_weight is None) != (k_weight is None):
+            raise KernelError("qkv_prepare_heads: the norm needs both weights or none")
     for t, name in ((q_weight, "q_weight"), (k_weight, "k_weight")):
         if t is not None:
             _need(t, name, torch.float32)
@@ -791,12 +829,13 @@ def qkv_prepare_heads(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_wei
             raise KernelError(f"qkv_prepare_heads: the rotary table has {cos_sin.shape[1]} pairs, {rot_dims} rotated dimensions want {rot_dims // 2}")
         n_positions = cos_sin.shape[0]
         _bounds("qkv_prepare_heads: row_pos", row_pos, n_positions, rows)
-    _bounds_paged("qkv_prepare_heads", rows, row_pos, row_slot, page_table, k_cache.shape[0])
+    if kv_heads > 0:
+        _bounds_paged("qkv_prepare_heads", rows, row_pos, row_slot, page_table, n_pages)
     _call(_fn("bc_qkv_prepare_heads_" + _suffix(q_out.dtype)), _ptr(qkv), _ptr(q_weight), _ptr(k_weight), _ptr(cos_sin if n_positions else None),
-          _c_int(n_positions), _ptr(row_pos), _ptr(row_slot), _ptr(page_table), _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]),
-          _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim),
-          _c_int(rot_dims if n_positions else 0), _c_int(pairing), _c_float(eps), _c_int(0 if q_weight is None else 1),
-          _c_int(1 if write_cache else 0), _stream())
+          _c_int(n_positions), _ptr(row_pos), _ptr(row_slot), _ptr(page_table), _c_int(page_table.shape[1]), _c_int(n_pages),
+          _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(value_heads), _c_int(head_dim),
+          _c_int(value_dim), _c_int(rot_dims if n_positions else 0), _c_int(pairing), _c_float(eps), _c_int(0 if q_weight is None else 1),
+          _c_int(1 if write_cache and kv_heads > 0 else 0), _stream())
 
 
 # ----------------------------------------------------------- recurrences with a decaying outer-product state
@@ -808,7 +847,7 @@ def linear_scan(q: torch.Tensor, q_at: int, q_rep: int, k: torch.Tensor, k_at: i
     """S_t = diag(a_t) S_(t-1) + (c_t k_t) v_t^T, o_t = out_scale * S_t^T q_t + skip * v_t for every head over every sequence's rows
     in time order, all float32.  q, k, v, decay and kscale are [rows, anything] tensors read from column ``*_at`` on: q and k hold
     ``key_dim`` values for each group of ``*_rep`` heads, v ``value_dim`` a head, decay ``key_dim`` a head (``vector_decay``) or one,
-    kscale one a head (None: 1).  ``state`` [slots, heads, value_dim, key_dim] (value channel by value channel), ``out`` [rows, heads * value_dim]."""
+    kscale one a head (None: 1).  A ``decay`` of a single row serves every row (constant decays).  ``state`` [slots, heads, value_dim, key_dim] (value channel by value channel), ``out`` [rows, heads * value_dim]."""
     for t, name in ((q, "q"), (k, "k"), (v, "v"), (decay, "decay"), (state, "state"), (out, "out")):
         _need(t, name, torch.float32)
     _need(seq_rows, "seq_rows", torch.int32)
@@ -819,7 +858,7 @@ def linear_scan(q: torch.Tensor, q_at: int, q_rep: int, k: torch.Tensor, k_at: i
         raise KernelError(f"linear_scan: state {tuple(state.shape)} or out {tuple(out.shape)} do not fit {H} heads of {N} x {P}")
     for t, at, width, name in ((q, q_at, H // q_rep * N, "q"), (k, k_at, H // k_rep * N, "k"), (v, v_at, H * P, "v"),
                                (decay, decay_at, H * N if vector_decay else H, "decay")):
-        if t.dim() != 2 or t.shape[0] < rows or at < 0 or at + width > t.shape[1]:
+        if t.dim() != 2 or (t.shape[0] < rows and not (t is decay and t.shape[0] == 1)) or at < 0 or at + width > t.shape[1]:
             raise KernelError(f"linear_scan: {name} {tuple(t.shape)} has no {width} columns from {at} on for {rows} rows")
     if kscale is not None:
         _need(kscale, "kscale", torch.float32)
@@ -836,7 +875,7 @@ def linear_scan(q: torch.Tensor, q_at: int, q_rep: int, k: torch.Tensor, k_at: i
         return _c_void_p(t.data_ptr() + 4 * col)
 
     _call(_fn("bc_linear_scan"), at(q, q_at), _c_int(q.shape[1]), _c_int(q_rep), at(k, k_at), _c_int(k.shape[1]), _c_int(k_rep), at(v, v_at),
-          _c_int(v.shape[1]), at(decay, decay_at), _c_int(decay.shape[1]), _c_int(1 if vector_decay else 0),
+          _c_int(v.shape[1]), at(decay, decay_at), _c_int(0 if decay.shape[0] == 1 else decay.shape[1]), _c_int(1 if vector_decay else 0),
           _c_void_p(0) if kscale is None else at(kscale, kscale_at), _c_int(0 if kscale is None else kscale.shape[1]), _ptr(skip),
           _c_float(out_scale), _ptr(state), _ptr(seq_rows), _ptr(seq_slot), _ptr(out), _c_int(seqs), _c_int(H), _c_int(N), _c_int(P),
           _c_int(state.shape[0]), _c_int(1 if write_state else 0), _stream())
@@ -845,21 +884,26 @@ def linear_scan(q: torch.Tensor, q_at: int, q_rep: int, k: torch.Tensor, k_at: i
 SSD_MAX_TAPS = 9
 
 
-def ssd_prepare(proj: torch.Tensor, conv_at: int, dt_at: int, weight_t: torch.Tensor, bias: Optional[torch.Tensor], dt_bias: torch.Tensor,
-                a_log: torch.Tensor, tail: torch.Tensor, seq_rows: torch.Tensor, seq_slot: torch.Tensor, xbc: torch.Tensor, dtda: torch.Tensor,
+def ssd_prepare(proj: torch.Tensor, conv_at: int, dt_at: int, weight_t: torch.Tensor, bias: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor],
+                a_log: Optional[torch.Tensor], tail: torch.Tensor, seq_rows: torch.Tensor, seq_slot: torch.Tensor, xbc: torch.Tensor,
+                dtda: Optional[torch.Tensor],
                 seqs: int, max_new: int, write_tail: bool = True) -> None:
     """xbc = silu(bias + causal convolution over time of proj's columns conv_at ..), channel by channel, with ``weight_t`` [taps, C]
     (the last tap is the current token's) and every slot's last taps - 1 inputs in ``tail`` [slots, taps - 1, C], brought up to date;
-    dtda[r] = (softplus(dt + dt_bias), exp(-exp(a_log) * that)) for the H step sizes at proj's columns dt_at ...  All float32."""
+    dtda[r] = (softplus(dt + dt_bias), exp(-exp(a_log) * that)) for the H step sizes at proj's columns dt_at .. (``dt_bias`` None: no
+    step sizes, the convolution alone).  All float32."""
     for t, name in ((proj, "proj"), (weight_t, "weight_t"), (dt_bias, "dt_bias"), (a_log, "a_log"), (tail, "tail"), (xbc, "xbc"), (dtda, "dtda")):
-        _need(t, name, torch.float32)
+        if dt_bias is not None or name not in ("dt_bias", "a_log", "dtda"):
+            _need(t, name, torch.float32)
     _need(seq_rows, "seq_rows", torch.int32)
     _need(seq_slot, "seq_slot", torch.int32)
     taps, C = weight_t.shape
-    H = dt_bias.numel()
+    H = 0 if dt_bias is None else dt_bias.numel()
     rows = proj.shape[0]
-    if a_log.numel() != H or tuple(xbc.shape) != (rows, C) or tuple(dtda.shape) != (rows, 2 * H) or conv_at + C > proj.shape[1] or dt_at + H > proj.shape[1]:
-        raise KernelError(f"ssd_prepare: proj {tuple(proj.shape)}, xbc {tuple(xbc.shape)}, dtda {tuple(dtda.shape)} do not fit {C} channels and {H} heads")
+    if H and (a_log.numel() != H or tuple(dtda.shape) != (rows, 2 * H)):
+        raise KernelError(f"ssd_prepare: a_log {a_log.numel()} or dtda {tuple(dtda.shape)} do not fit {H} heads")
+    if tuple(xbc.shape) != (rows, C) or conv_at + C > proj.shape[1] or dt_at + H > proj.shape[1]:
+        raise KernelError(f"ssd_prepare: proj {tuple(proj.shape)}, xbc {tuple(xbc.shape)} do not fit {C} channels and {H} heads")
     if tuple(tail.shape[1:]) != (max(taps - 1, 1), C) or not 1 <= taps <= SSD_MAX_TAPS:
         raise KernelError(f"ssd_prepare: tail {tuple(tail.shape)} does not fit {taps} taps of {C} channels (at most {SSD_MAX_TAPS} taps)")
     if bias is not None:
@@ -886,11 +930,13 @@ def gla_decay(proj: torch.Tensor, inner_at: int, w2t: torch.Tensor, bias: torch.
 
 
 def gated_norm(y: torch.Tensor, gate: torch.Tensor, gate_at: int, weight: torch.Tensor, out: torch.Tensor, parts: int, eps: float,
-               gate_first: bool, factor: float = 1.0, row_slot: Optional[torch.Tensor] = None) -> None:
+               gate_first: bool, factor: float = 1.0, row_slot: Optional[torch.Tensor] = None, activation: str = "silu") -> None:
     """Every row of y [rows, W] (float32) in ``parts`` equal parts, each divided by its own root mean square and multiplied by
-    ``weight`` (as wide as the row, or as a part and then shared by the parts); silu of the gate (columns gate_at .. of ``gate``,
+    ``weight`` (as wide as the row, or as a part and then shared by the parts); silu (or ``activation`` "sigmoid") of the gate (columns gate_at .. of ``gate``,
     float32) multiplies before the norm (``gate_first``) or after it; ``factor`` multiplies the result.  With ``row_slot``, rows whose
     slot is negative are not read and give zeros."""
+    if activation not in ("silu", "sigmoid"):
+        raise KernelError(f"gated_norm: a gate is 'silu' or 'sigmoid', not {activation!r}")
     _need(y, "y", torch.float32)
     _need(gate, "gate", torch.float32)
     _need(weight, "weight", torch.float32)
@@ -904,7 +950,202 @@ def gated_norm(y: torch.Tensor, gate: torch.Tensor, gate_at: int, weight: torch.
             raise KernelError("gated_norm: fewer slots than rows")
     _call(_fn("bc_gated_norm_" + _suffix(out.dtype)), _ptr(y), _c_void_p(gate.data_ptr() + 4 * gate_at), _c_int(gate.shape[1]), _ptr(weight),
           _c_int(weight.numel()), _ptr(row_slot), _ptr(out), _c_int(rows), _c_int(W), _c_int(parts), _c_float(eps), _c_int(1 if gate_first else 0),
-          _c_float(factor), _stream())
+          _c_int(1 if activation == "sigmoid" else 0), _c_float(factor), _stream())
+
+
+# ------------------------------------------------------------- a residual stream of several copies
+
+HYPER_MAX_STREAMS = 64
+
+
+def hyper_start(e: torch.Tensor, weight: Optional[torch.Tensor], x: torch.Tensor, eps: float) -> None:
+    """x[r, s] = e[r] / rms(e[r]) * weight for every stream s (``weight`` None: e as it is); x [rows, S, E], e [rows, E], float32."""
+    _need(e, "e", torch.float32)
+    _need(x, "x", torch.float32)
+    rows, S, E = x.shape
+    if tuple(e.shape) != (rows, E):
+        raise KernelError(f"hyper_start: e {tuple(e.shape)} does not fit x {tuple(x.shape)}")
+    if weight is not None:
+        _need(weight, "weight", torch.float32)
+        if weight.numel() != E:
+            raise KernelError(f"hyper_start: a weight of {weight.numel()} for rows of {E}")
+    _call(_fn("bc_hyper_start"), _ptr(e), _ptr(weight), _ptr(x), _c_int(rows), _c_int(S), _c_int(E), _c_float(eps), _stream())
+
+
+def hyper_step(x: torch.Tensor, y: Optional[torch.Tensor], scale: Optional[torch.Tensor], mix: Optional[torch.Tensor], out_w: Optional[torch.Tensor],
+               in_w: Optional[torch.Tensor], weight: torch.Tensor, h: torch.Tensor, eps: float, gather: Optional[torch.Tensor] = None) -> None:
+    """Between two sublayers of a row's bundle x [rows, S, E] (float32): with a pending result ``y`` [rows, E],
+    x[t] <- sum_s mix[s, t] x[s] + out_w[t] * scale * y and y <- 0; then u = sum_t in_w[t] x[t] (``in_w`` None: ones) and
+    h = u / rms(u) * weight in h's type.  With ``gather`` only the rows it names are taken and x and y stay as they are."""
+    _need(x, "x", torch.float32)
+    _need(weight, "weight", torch.float32)
+    _need(h, "h")
+    x_rows, S, E = x.shape
+    rows = h.shape[0]
+    if h.shape[-1] != E or weight.numel() != E:
+        raise KernelError(f"hyper_step: h {tuple(h.shape)} or a weight of {weight.numel()} do not fit x {tuple(x.shape)}")
+    for t, name, n in ((y, "y", x_rows * E), (scale, "scale", E), (mix, "mix", S * S), (out_w, "out_w", S), (in_w, "in_w", S)):
+        if t is not None:
+            _need(t, name, torch.float32)
+            if t.numel() != n:
+                raise KernelError(f"hyper_step: {name} has {t.numel()} values, wanted {n}")
+    if gather is not None:
+        _need(gather, "gather", torch.int32)
+        if gather.numel() != rows:
+            raise KernelError("hyper_step: gather and h differ in rows")
+        _bounds("hyper_step: gather", gather, x_rows)
+    elif rows != x_rows:
+        raise KernelError("hyper_step: x and h differ in rows")
+    _call(_fn("bc_hyper_step_" + _suffix(h.dtype)), _ptr(x), _ptr(y), _ptr(scale), _ptr(mix), _ptr(out_w), _ptr(in_w), _ptr(weight), _ptr(gather), _ptr(h),
+          _c_int(rows), _c_int(x_rows), _c_int(S), _c_int(E), _c_float(eps), _stream())
+
+
+# ------------------------------------------------------ the delta rule with a decay a key channel
+
+def delta_split(proj: torch.Tensor, at0: int, out0: torch.Tensor, at1: int, out1: torch.Tensor, terms: int) -> None:
+    """Columns at0 .. and at1 .. of proj (float32) as rows of their own: ``terms`` 1 copies them into float32 outputs, 2 writes bf16 rows
+    [hi | lo] with hi + lo the value to about 2^-17."""
+    _need(proj, "proj", torch.float32)
+    for t in (out0, out1):
+        _need(t, "out", torch.bfloat16 if terms == 2 else torch.float32)
+        if t.shape[0] != proj.shape[0] or t.shape[1] % terms:
+            raise KernelError(f"delta_split: out {tuple(t.shape)} does not fit proj {tuple(proj.shape)}")
+    _call(_fn("bc_delta_split"), _ptr(proj), _c_int(proj.shape[1]), _c_int(at0), _c_int(out0.shape[1] // terms), _ptr(out0), _c_int(at1),
+          _c_int(out1.shape[1] // terms), _ptr(out1), _c_int(1 if terms == 2 else 0), _c_int(proj.shape[0]), _stream())
+
+
+def delta_channel_prepare(qkv: torch.Tensor, z: torch.Tensor, proj: torch.Tensor, b_at: int, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                          scal: torch.Tensor, heads: int, kv_heads: int, head_dim: int) -> None:
+    """In place: q and k at the front of qkv's rows become unit vectors a head (q over sqrt(head_dim) too), z [rows, heads * head_dim] the
+    decays exp(-exp(a_log) softplus(z + dt_bias)); scal [rows, heads, 2] = (sigmoid of proj's columns b_at .., q . k).  All float32."""
+    for t, name in ((qkv, "qkv"), (z, "z"), (proj, "proj"), (a_log, "a_log"), (dt_bias, "dt_bias"), (scal, "scal")):
+        _need(t, name, torch.float32)
+    rows, H, G, D = qkv.shape[0], heads, kv_heads, head_dim
+    if tuple(z.shape) != (rows, H * D) or tuple(scal.shape) != (rows, H, 2) or proj.shape[0] != rows or a_log.numel() != H or dt_bias.numel() != H * D:
+        raise KernelError(f"delta_channel_prepare: z {tuple(z.shape)}, scal {tuple(scal.shape)} do not fit {H} heads of {D}")
+    _call(_fn("bc_delta_channel_prepare"), _ptr(qkv), _c_int(qkv.shape[1]), _ptr(z), _ptr(proj), _c_int(proj.shape[1]), _c_int(b_at), _ptr(a_log),
+          _ptr(dt_bias), _ptr(scal), _c_int(rows), _c_int(H), _c_int(G), _c_int(D), _stream())
+
+
+def _delta_channel_check(who: str, qkv, state, out, rows: int, H: int, G: int, D: int, P: int) -> None:
+    if tuple(state.shape[1:]) != (H, P, D) or tuple(out.shape) != (rows, H * P) or qkv.shape[1] < 2 * G * D + H * P or H % G:
+        raise KernelError(f"{who}: qkv {tuple(qkv.shape)}, state {tuple(state.shape)} or out {tuple(out.shape)} do not fit {H} heads on {G} of {D} x {P}")
+
+
+def delta_channel_scan(qkv: torch.Tensor, decay: torch.Tensor, scal: torch.Tensor, state: torch.Tensor, seq_rows: torch.Tensor, seq_slot: torch.Tensor,
+                       out: torch.Tensor, seqs: int, heads: int, kv_heads: int, head_dim: int, value_dim: int, write_state: bool = True) -> None:
+    """S <- diag(decay) S; r = b (v - S^T k); S <- S + k r^T; o = S^T q over every sequence's rows in time order, from and into ``state``
+    [slots, heads, value_dim, head_dim] float32; qkv [rows, 2 kv_heads head_dim + heads value_dim] and scal as delta_channel_prepare leaves them."""
+    for t, name in ((qkv, "qkv"), (decay, "decay"), (scal, "scal"), (state, "state"), (out, "out")):
+        _need(t, name, torch.float32)
+    _need(seq_rows, "seq_rows", torch.int32)
+    _need(seq_slot, "seq_slot", torch.int32)
+    _delta_channel_check("delta_channel_scan", qkv, state, out, qkv.shape[0], heads, kv_heads, head_dim, value_dim)
+    if tuple(decay.shape) != (qkv.shape[0], heads * head_dim) or tuple(scal.shape) != (qkv.shape[0], heads, 2):
+        raise KernelError("delta_channel_scan: decay or scal do not fit")
+    _bounds("delta_channel_scan: seq_slot", seq_slot, state.shape[0], seqs, lowest=-1)
+    _bounds("delta_channel_scan: seq_rows", seq_rows, qkv.shape[0] + 1, seqs + 1)
+    _call(_fn("bc_delta_channel_scan"), _ptr(qkv), _c_int(qkv.shape[1]), _ptr(decay), _ptr(scal), _ptr(state), _ptr(seq_rows), _ptr(seq_slot), _ptr(out),
+          _c_int(seqs), _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim), _c_int(state.shape[0]), _c_int(1 if write_state else 0), _stream())
+
+
+def delta_channel_step_accepts(head_dim: int, value_dim: int, decay_rank: int, gate_rank: int) -> bool:
+    """Whether the one-launch step for single rows takes these sizes."""
+    return 0 < head_dim <= 256 and 0 < value_dim <= 2048 and 0 < decay_rank <= 2048 and 0 < gate_rank <= 2048
+
+
+def delta_channel_step(qkv: torch.Tensor, proj: torch.Tensor, b_at: int, a_at: int, g_at: int, w_a2: torch.Tensor, w_g2: torch.Tensor, a_log: torch.Tensor,
+                       dt_bias: torch.Tensor, norm_weight: torch.Tensor, state: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor, heads: int,
+                       kv_heads: int, head_dim: int, value_dim: int, eps: float, write_state: bool = True) -> None:
+    """A step in which every sequence brings one row (row r lives in slot ``row_slot[r]``): decays and gates from the inner vectors at
+    proj's columns a_at and g_at, unit q and k from the convolved ones in qkv, one step of the recurrence, the norm over each head's
+    values times ``norm_weight`` and the gate; out [rows, heads * value_dim] in the type of ``w_a2``."""
+    for t, name in ((qkv, "qkv"), (proj, "proj"), (a_log, "a_log"), (dt_bias, "dt_bias"), (norm_weight, "norm_weight"), (state, "state")):
+        _need(t, name, torch.float32)
+    _need(row_slot, "row_slot", torch.int32)
+    _need(out, "out")
+    _need(w_a2, "w_a2", out.dtype)
+    _need(w_g2, "w_g2", out.dtype)
+    rows, H, G, D, P = qkv.shape[0], heads, kv_heads, head_dim, value_dim
+    _delta_channel_check("delta_channel_step", qkv, state, out, rows, H, G, D, P)
+    ra, rg = w_a2.shape[1], w_g2.shape[1]
+    if w_a2.shape[0] != H * D or w_g2.shape[0] != H * P or a_log.numel() != H or dt_bias.numel() != H * D or norm_weight.numel() != P \
+            or max(a_at + ra, g_at + rg, b_at + H) > proj.shape[1] or row_slot.numel() < rows or proj.shape[0] < rows:
+        raise KernelError(f"delta_channel_step: w_a2 {tuple(w_a2.shape)}, w_g2 {tuple(w_g2.shape)} or proj {tuple(proj.shape)} do not fit")
+    _bounds("delta_channel_step: row_slot", row_slot, state.shape[0], rows, lowest=-1)
+    _call(_fn("bc_delta_channel_step_" + _suffix(out.dtype)), _ptr(qkv), _c_int(qkv.shape[1]), _ptr(proj), _c_int(proj.shape[1]), _c_int(b_at), _c_int(a_at),
+          _c_int(ra), _c_int(g_at), _c_int(rg), _ptr(w_a2), _ptr(w_g2), _ptr(a_log), _ptr(dt_bias), _ptr(norm_weight), _ptr(state), _ptr(row_slot), _ptr(out),
+          _c_int(rows), _c_int(H), _c_int(G), _c_int(D), _c_int(P), _c_float(eps), _c_int(state.shape[0]), _c_int(1 if write_state else 0), _stream())
+
+
+# ------------------------------------------------------------------------ differential attention
+
+def _diff_check(who: str, q, k_cache, v_cache, page_table, out, H: int, G: int, D: int, DV: int) -> None:
+    _need(q, "q")
+    _need(k_cache, "k_cache", q.dtype)
+    _need(v_cache, "v_cache", q.dtype)
+    _need(page_table, "page_table", torch.int32)
+    _need(out, "out", q.dtype)
+    rows = q.shape[0]
+    if tuple(q.shape) != (rows, H * 2 * D) or tuple(out.shape) != (rows, H * DV) or tuple(k_cache.shape[1:]) != (2 * G, PAGE, D) \
+            or tuple(v_cache.shape) != (k_cache.shape[0], G, PAGE, DV):
+        raise KernelError(f"{who}: q {tuple(q.shape)}, out {tuple(out.shape)}, cache {tuple(k_cache.shape)} and {tuple(v_cache.shape)} do not fit {H} heads on "
+                          f"{G} of two maps of {D} and values of {DV}")
+
+
+def diff_rows(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, row_pos: torch.Tensor, row_slot: torch.Tensor,
+              out: torch.Tensor, heads: int, kv_heads: int, head_dim: int, value_dim: int, window: int, keep_first: int, scale: float, lam: float,
+              eps: float, factor: float) -> None:
+    """Differential attention, one warp a (row, head): q [rows, heads * 2 * head_dim] head by head [map 0 | map 1], k_cache [pages,
+    2 kv_heads, 64, head_dim], v_cache [pages, kv_heads, 64, value_dim]; a row at position i sees j <= i with i - j < window or
+    j < keep_first (window 0: all).  out = (A_0 - lam A_1) over its root mean square, times ``factor``."""
+    _diff_check("diff_rows", q, k_cache, v_cache, page_table, out, heads, kv_heads, head_dim, value_dim)
+    _need(row_pos, "row_pos", torch.int32)
+    _need(row_slot, "row_slot", torch.int32)
+    _bounds_paged("diff_rows", q.shape[0], row_pos, row_slot, page_table, k_cache.shape[0])
+    _call(_fn("bc_diff_rows_" + _suffix(q.dtype)), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(row_pos), _ptr(row_slot), _ptr(out),
+          _c_int(q.shape[0]), _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim), _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]),
+          _c_int(window), _c_int(keep_first), _c_float(scale), _c_float(lam), _c_float(eps), _c_float(factor), _stream())
+
+
+def diff_tiles_accepts(heads: int, kv_heads: int, head_dim: int, value_dim: int, dtype: torch.dtype) -> bool:
+    """Whether the tensor-core tile kernel takes these sizes (bf16, widths multiples of 8: maps up to 128, values up to 256)."""
+    return dtype == torch.bfloat16 and bool(_fn("bc_diff_tiles_accepts")(_c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim)))
+
+
+def diff_tiles_splits(seqs: int, kv_heads: int, reach: int, window: int, keep_first: int) -> int:
+    """Blocks that share a row's pages in steps of one row a sequence: about two a multiprocessor in all, never more than there are
+    pages (``reach``: a bound on the positions any row reaches; a window bounds them further)."""
+    pages = -(-max(reach, 1) // PAGE)
+    if window > 0:
+        pages = min(pages, -(-keep_first // PAGE) + (window + PAGE - 2) // PAGE + 1)
+    return max(1, min(pages, 2 * sm_count() // max(seqs * kv_heads, 1), 65535 // max(seqs, 1)))
+
+
+def diff_tiles(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, seq_rows: torch.Tensor, seq_slot: torch.Tensor,
+               seq_start: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor, seqs: int, max_new: int, heads: int, kv_heads: int, head_dim: int,
+               value_dim: int, window: int, keep_first: int, scale: float, lam: float, eps: float, factor: float, splits: int = 1) -> None:
+    """What diff_rows computes, for bf16 on tensor-core tiles; sequence s brings rows seq_rows[s] .. seq_rows[s + 1] and held seq_start[s]
+    positions before.  ``splits`` > 1 shares the pages a block would walk out over that many blocks, merged in their order."""
+    _diff_check("diff_tiles", q, k_cache, v_cache, page_table, out, heads, kv_heads, head_dim, value_dim)
+    _need(q, "q", torch.bfloat16)
+    for t, name in ((seq_rows, "seq_rows"), (seq_slot, "seq_slot"), (seq_start, "seq_start"), (row_slot, "row_slot")):
+        _need(t, name, torch.int32)
+    rows = q.shape[0]
+    if seq_rows.numel() < seqs + 1 or seq_slot.numel() < seqs or seq_start.numel() < seqs or row_slot.numel() < rows:
+        raise KernelError("diff_tiles: fewer sequence entries than sequences")
+    _bounds("diff_tiles: seq_slot", seq_slot, page_table.shape[0], seqs, lowest=-1)
+    _bounds("diff_tiles: seq_rows", seq_rows, rows + 1, seqs + 1)
+    _bounds("diff_tiles: page_table", page_table, k_cache.shape[0], lowest=-1)
+    global launches
+    scratch = None
+    if splits > 1:
+        scratch, _ = _decode_workspace(q.device, rows * heads * splits * 2 * (value_dim + 2), 1)
+        launches += 1        # the merge
+    _call(_fn("bc_diff_tiles_bf16"), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(seq_rows), _ptr(seq_slot), _ptr(seq_start), _ptr(row_slot),
+          _ptr(out), _ptr(scratch), _c_int(splits), _c_int(rows), _c_int(seqs), _c_int(max_new), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
+          _c_int(value_dim), _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_int(keep_first), _c_float(scale), _c_float(lam),
+          _c_float(eps), _c_float(factor), _stream())
 
 
 # ---------------------------------------------------------------------- attention whose heads talk

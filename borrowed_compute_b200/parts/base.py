@@ -10,6 +10,8 @@ A model is put together from parts that know nothing of the model they are in:
 - a *short convolution* mixes a few neighbouring rows of one sequence on every channel and
   keeps the last of them as per-sequence state;
 - a *block* arranges norms, a mixer and a feed-forward around the residual stream;
+- a *connection* and a *channel scale* stand around a sublayer where a row's residual stream is a
+  bundle of several copies (``parts/streams.py``);
 - a *junction* acts on the residual stream between two layers (where a stretch of layers is
   entered again, say) and may read the embedding's output.
 
@@ -66,6 +68,8 @@ POSITION_ENCODINGS = Registry("position encoding")
 CONVOLUTIONS = Registry("short convolution")
 BLOCKS = Registry("block")
 JUNCTIONS = Registry("junction")
+CONNECTIONS = Registry("connection")
+SCALES = Registry("channel scale")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
 
@@ -133,6 +137,10 @@ class ModelSpec:
     tolerated: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()
     # Parts that act on the stream between layers; a RunSpec's ``enter`` names one.
     junctions: Tuple[PartSpec, ...] = ()
+    # A norm of the embedded rows before they enter the stream (or None).
+    embedding_norm: Optional[PartSpec] = None
+    # Copies of the residual stream a row carries: 0, one plain stream; else the blocks are handed a StreamBundle of that many.
+    streams: int = 0
 
 
 # -------------------------------------------------------------------------- declared tensors
@@ -200,6 +208,13 @@ class CacheNeed:
 
     def key(self) -> Tuple:
         return (self.planes, self.window, self.chunk, self.keep_first)
+
+    def widened(self, other: "CacheNeed") -> "CacheNeed":
+        """What serves this need and ``other`` (of a run that reads the same memory) alike: every position either of them reads is kept."""
+        if self.planes != other.planes:
+            raise ValueError(f"a run cannot read planes {other.planes} out of memory with planes {self.planes}")
+        return CacheNeed(self.planes, window=max(self.window, other.window) if self.window and other.window else 0,
+                         chunk=self.chunk if self.chunk == other.chunk else 0, keep_first=max(self.keep_first, other.keep_first))
 
     def values_per_token(self) -> int:
         return sum(h * w for h, w in self.planes)
@@ -390,6 +405,8 @@ class Block(Part):
     those of ``OPTIONAL``, which a layer may leave out (the attribute is then None).  The
     built parts are attributes of the block under their role names."""
 
+    # True for blocks whose forward takes a StreamBundle instead of one residual tensor (ModelSpec.streams > 0).
+    STREAMS = False
     ROLES: Dict[str, Registry] = {}
     OPTIONAL: Tuple[str, ...] = ()
 

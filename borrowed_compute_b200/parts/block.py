@@ -10,7 +10,10 @@ without a norm of its own reads what the mixer reads, x += mixer(h) + feed_forwa
 h = norm1(x).
 
 The sandwich block: a norm before and after each sublayer, x += norm1b(mixer(conv(norm1(x)))); x += norm2b(ff(norm2(x))).
-The second half may be left out, and so may the short convolution (or token shift) of the mixer's input."""
+The second half may be left out, and so may the short convolution (or token shift) of the mixer's input.
+
+The hyper-connected block: a pre-norm block on a bundle of streams (``parts/streams.py``), each sublayer between the two ends of its
+connection, its result scaled channel by channel.  The feed-forward and what belongs to it may be left out, and so may the scales."""
 
 from __future__ import annotations
 
@@ -21,7 +24,8 @@ from typing import Dict, Mapping
 from .. import ops
 from .norm import RMSNorm
 from .short_conv import CausalConvResidual
-from .base import BLOCKS, CONVOLUTIONS, FEED_FORWARDS, MIXERS, NORMS, Block, RunMemory, Runtime, StateNeed, StepContext
+from .streams import StreamBundle
+from .base import BLOCKS, CONNECTIONS, CONVOLUTIONS, FEED_FORWARDS, MIXERS, NORMS, SCALES, Block, RunMemory, Runtime, StateNeed, StepContext
 
 
 @BLOCKS.register("prenorm")
@@ -145,3 +149,27 @@ class SandwichBlock(Block):
                 self.norm2.forward(residual, h)
             self.feed_forward.forward(h, y, ctx)
             ops.norm_add(y, self.norm2b.weight, residual, self.norm2b.eps)
+
+
+@BLOCKS.register("hyper_connected")
+class HyperConnectedBlock(Block):
+    STREAMS = True
+    ROLES = {"norm1": NORMS, "mixer": MIXERS, "scale1": SCALES, "connection1": CONNECTIONS, "norm2": NORMS, "feed_forward": FEED_FORWARDS,
+             "scale2": SCALES, "connection2": CONNECTIONS}
+    OPTIONAL = ("scale1", "norm2", "feed_forward", "scale2", "connection2")
+
+    def __init__(self, parts, hidden_size: int):
+        super().__init__(parts, hidden_size)
+        if len({self.norm2 is None, self.feed_forward is None, self.connection2 is None}) != 1 or (self.scale2 is not None and self.feed_forward is None):
+            raise ValueError("a hyper-connected block has a feed-forward with its norm and connection, or none of the three")
+        for role in ("norm1", "norm2"):
+            if getattr(self, role) is not None and type(getattr(self, role)) is not RMSNorm:
+                raise ValueError(f"the norm of a collapsed bundle ('{role}') must be an RMS norm")
+
+    def forward(self, bundle: StreamBundle, ctx: StepContext, mem: RunMemory, rt: Runtime) -> None:
+        h = torch.empty(bundle.y.shape, dtype=rt.dtype, device=bundle.y.device)
+        self.mixer.forward(h, bundle.enter(self.connection1, self.norm1, h), ctx, mem)
+        bundle.leave(self.connection1, self.scale1)
+        if self.feed_forward is not None:
+            self.feed_forward.forward(h, bundle.enter(self.connection2, self.norm2, h), ctx)
+            bundle.leave(self.connection2, self.scale2)

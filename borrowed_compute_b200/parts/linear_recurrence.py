@@ -3,7 +3,7 @@
     S_t = diag(a_t) S_(t-1) + (c_t k_t) v_t^T          o_t = f S_t^T q_t + d v_t
 
 per head, S being [key channels, value channels], zero at a sequence's start and carried from token to
-token in the cache's per-sequence state.  Two mixers are this recurrence (``csrc/linear_scan.cu`` runs it,
+token in the cache's per-sequence state.  Three mixers are this recurrence (``csrc/linear_scan.cu`` runs it,
 the same kernel for prompts and single rows, so that both give the same bits):
 
 ``gated_linear_attention``: q, k (heads x dim) and v (heads x vdim) from h; a decay per key channel
@@ -14,6 +14,9 @@ mean square times a weight of vdim values shared by the heads, times silu(W_g h)
 with bias and silu whose last inputs are per-sequence state too; dt = softplus(dt + dt_bias), a = exp(-exp(A_log) dt)
 one number a head, c = dt, k = B and q = C of the head's group, v = x, d = D.  The heads' outputs times silu(z), then
 an RMS norm in ``norm_groups`` equal parts times a weight, then W_o.
+
+``lightning_attention``: q, k = silu(W h) (heads x dim), v = silu(W_v h) (heads x vdim); a one constant a head; c = f = 1, d = 0.  The
+heads' outputs side by side over their common root mean square times a weight, times sigmoid(W_g h), then W_o.
 
 The projections keep their float accumulators; decays, step sizes, gates, norms and the state are float on both
 paths.  ``out_scale`` multiplies the mixer's result (a mixer that runs beside another).
@@ -77,6 +80,47 @@ class GatedLinearAttention(Mixer):
                         ctx.seq_slot, o, ctx.seqs, H, D, P, write_state=mem.writes)
         y = torch.empty((rows, hp), dtype=x.dtype, device=dev)
         ops.gated_norm(o, proj, 2 * hd + hp, self.norm_weight, y, H, self.norm_eps, gate_first=False, factor=self.out_scale, row_slot=ctx.row_slot)
+        products.linear(y, self.w_o, residual, products.EPI_ADD_F32, "output product")
+
+
+@MIXERS.register("lightning_attention")
+class LightningAttention(Mixer):
+    def __init__(self, hidden_size: int, heads: int, head_dim: int, value_dim: int, decay, norm_eps: float):
+        super().__init__(hidden_size=hidden_size, heads=heads, head_dim=head_dim, value_dim=value_dim, decay=decay, norm_eps=norm_eps)
+        if not 0 < int(head_dim) <= 256:
+            raise ValueError(f"a head of {head_dim} key channels is outside what the recurrence kernel takes (1 to 256)")
+        self.hidden_size, self.heads, self.head_dim, self.value_dim = int(hidden_size), int(heads), int(head_dim), int(value_dim)
+        self.decay, self.norm_eps = tuple(float(d) for d in decay), float(norm_eps)
+        if len(self.decay) != self.heads:
+            raise ValueError(f"{len(self.decay)} decays for {heads} heads")
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        e, hd, hp = self.hidden_size, self.heads * self.head_dim, self.heads * self.value_dim
+        return {"q": TensorSpec((hd, e)), "k": TensorSpec((hd, e)), "v": TensorSpec((hp, e)), "g": TensorSpec((hp, e)),
+                "norm": TensorSpec((hp,), role="vector", init="ones"), "o": TensorSpec((e, hp))}
+
+    def state_need(self) -> Optional[StateNeed]:
+        return StateNeed((self.heads, self.value_dim, self.head_dim), torch.float32)      # value channel by value channel
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        super().load(tensors, rt)
+        self.w_in = torch.cat([tensors[n] for n in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.w_o, self.norm_weight = tensors["o"].contiguous(), tensors["norm"].contiguous()
+        self.decays = torch.tensor([self.decay], dtype=torch.float32, device=self.w_in.device)      # one row that every token reads
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext, mem: RunMemory) -> None:
+        if mem.state is None:
+            raise RuntimeError("lightning attention was given no state: the cache does not serve this run")
+        rows, H, D, P, dev = x.shape[0], self.heads, self.head_dim, self.value_dim, x.device
+        hd, hp = H * D, H * P
+        proj = torch.empty((rows, self.w_in.shape[0]), dtype=torch.float32, device=dev)
+        # q, k and v leave the product's epilogue through silu, the gate as it is.
+        products.linear(x, self.w_in, proj, products.EPI_SILU_F32, "recurrence projections", cols=2 * hd + hp)
+        o = torch.empty((rows, hp), dtype=torch.float32, device=dev)
+        ops.linear_scan(proj, 0, 1, proj, hd, 1, proj, 2 * hd, self.decays, 0, False, None, 0, None, 1.0, mem.state, ctx.seq_rows, ctx.seq_slot, o,
+                        ctx.seqs, H, D, P, write_state=mem.writes)
+        y = torch.empty((rows, hp), dtype=x.dtype, device=dev)
+        ops.gated_norm(o, proj, 2 * hd + hp, self.norm_weight, y, 1, self.norm_eps, gate_first=False, row_slot=ctx.row_slot, activation="sigmoid")
         products.linear(y, self.w_o, residual, products.EPI_ADD_F32, "output product")
 
 

@@ -43,13 +43,19 @@ class SwiGLU(FeedForward):
 
 @FEED_FORWARDS.register("plain_mlp")
 class PlainMLP(FeedForward):
-    """down( act(up x) ) without a gate; ``activation``: "relu2", the square of relu, applied to the up product's float sums in its
-    epilogue and rounded once.  ``up`` and ``down`` are the names the matrices carry after the part's prefix."""
+    """down( act(up x) ) without a gate; the activation is applied to the up product's float sums in its epilogue and rounded once:
 
-    ACTIVATIONS = ("relu2",)
+    - "relu2", the square of relu;
+    - "xielu", with two learned numbers p and q (tensor ``act``): softplus(p) z^2 + z/2 above zero,
+      (1/2 + softplus(q)) (e^z - 1 - z) + z/2 below.
 
-    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu2", up: str = "up", down: str = "down"):
-        super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, activation=activation, up=up, down=down)
+    ``up``, ``down`` and ``act`` are the names the tensors carry after the part's prefix."""
+
+    ACTIVATIONS = ("relu2", "xielu")
+
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu2", up: str = "up", down: str = "down", act: str = "act"):
+        super().__init__(hidden_size=hidden_size, intermediate_size=intermediate_size, activation=activation, up=up, down=down, act=act)
+        self.act = str(act)
         if activation not in self.ACTIVATIONS:
             raise ValueError(f"activation {activation!r} is not known (known: {list(self.ACTIVATIONS)})")
         self.hidden_size, self.intermediate_size, self.activation = int(hidden_size), int(intermediate_size), activation
@@ -57,15 +63,22 @@ class PlainMLP(FeedForward):
 
     def tensors(self) -> Dict[str, TensorSpec]:
         e, f = self.hidden_size, self.intermediate_size
-        return {self.names[0]: TensorSpec((f, e)), self.names[1]: TensorSpec((e, f))}
+        out = {self.names[0]: TensorSpec((f, e)), self.names[1]: TensorSpec((e, f))}
+        if self.activation == "xielu":
+            out[self.act] = TensorSpec((2,), role="vector", init="zeros")
+        return out
 
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         super().load(tensors, rt)
         self.w_up, self.w_down = tensors[self.names[0]].contiguous(), tensors[self.names[1]].contiguous()
+        self.numbers = None
+        if self.activation == "xielu":
+            p, q = torch.nn.functional.softplus(tensors[self.act].double()).tolist()       # of the weights alone: once
+            self.numbers = (p, 0.5 + q)
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:
         act = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
-        products.linear(x, self.w_up, act, products.EPI_RELU2, "up product")
+        products.linear(x, self.w_up, act, products.EPI_RELU2 if self.numbers is None else products.EPI_XIELU, "up product", act=self.numbers)
         products.linear(act, self.w_down, residual, products.EPI_ADD_F32, "down product")
 
 
