@@ -925,6 +925,91 @@ def bench_logirax(pk, rng, size="wide", layers=4, batch=8, prompt=PROMPT, steps=
     return _bench_models(configs, costs_of, c["vocab"], out, pk, rng, FP32_TFLOPS, batch, prompt, steps, warmup)
 
 
+# -------------------------------------------------------------------- the sixth architecture
+DURATAR_SIZES = {
+    # the width, projections and feed-forward of the 8B shape: 32 heads of two maps of 64 on values of 128, delta heads and lightning heads that
+    # fill the width, four streams
+    "wide": dict(width=4096, heads=32, kv_heads=8, dim=64, vdim=128, window=1024, keep=4, delta_heads=64, delta_dim=64, delta_vdim=64, rank=64,
+                 light_heads=32, light_dim=128, light_vdim=128, ff=14336, streams=4, vocab=32000),
+    # a 2,048-wide model, values as wide as a map
+    "mid": dict(width=2048, heads=16, kv_heads=4, dim=64, vdim=64, window=512, keep=4, delta_heads=32, delta_dim=64, delta_vdim=64, rank=32,
+                light_heads=16, light_dim=128, light_vdim=128, ff=8192, streams=4, vocab=32000),
+}
+
+
+def duratar_config(width, heads, kv_heads, dim, vdim, window, keep, delta_heads, delta_dim, delta_vdim, rank, light_heads, light_dim, light_vdim, ff, streams,
+                   vocab, layers):
+    """``layers`` layers of the Duratar design in turns of four: the delta rule, attention, lightning, attention over the first one's keys and values."""
+    out = []
+    for i in range(layers):
+        attention = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window, "keep_first": keep}, "diff": 0.4,
+                     "rot": {"dims": dim // 2, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}, "scale": 1.0 / dim ** 0.5}
+        if i % 4 == 0:
+            mixer, kind = {"heads": delta_heads, "kv_heads": delta_heads, "dim": delta_dim, "vdim": delta_vdim, "conv": 4, "decay_rank": rank, "gate_rank": rank}, "channel_delta"
+        elif i % 4 == 2:
+            mixer, kind = {"heads": light_heads, "dim": light_dim, "vdim": light_vdim, "decay": [1.0 - 2.0 ** (-3 - 6 * h / light_heads) for h in range(light_heads)]}, "lightning"
+        else:
+            mixer, kind = dict(attention, kv_from=i - 2) if i % 4 == 3 else attention, "attention"
+        out.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Duratar", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": 1e-5}, "layers": out}
+
+
+def duratar_costs(c, layers, batch, ctx_len, T) -> dict:
+    """What each kernel class of the Duratar model has to move in a decode step (bytes) and to compute in a prompt step of T tokens
+    (operations, or bytes where it only moves data), summed over the model's layers."""
+    E, H, G, D, DV, W, K, S, F, V, B = (c["width"], c["heads"], c["kv_heads"], c["dim"], c["vdim"], c["window"], c["keep"], c["streams"], c["ff"], c["vocab"], batch)
+    Hd, Dd, Pd, rank, Hl, Dl, Pl = c["delta_heads"], c["delta_dim"], c["delta_vdim"], c["rank"], c["light_heads"], c["light_dim"], c["light_vdim"]
+    nd, nl = sum(i % 4 == 0 for i in range(layers)), sum(i % 4 == 2 for i in range(layers))
+    na, nq = sum(i % 4 == 1 for i in range(layers)), sum(i % 4 == 3 for i in range(layers))
+    ch = 2 * Hd * Dd + Hd * Pd
+    n_d, n_l, n_q = ch + 2 * rank + Hd, 2 * Hl * Dl + 2 * Hl * Pl, 2 * H * D
+    n_qkv = n_q + 2 * G * D + G * DV
+    seen = lambda t: min(t + 1, W) + max(0, min(K, t + 1 - W))                                                       # noqa: E731
+    seen_decode, seen_prefill = seen(ctx_len), sum(seen(t) for t in range(T))
+    state_d, state_l = Hd * Dd * Pd * 4.0, Hl * Dl * Pl * 4.0
+    mul = lambda n, k, out: 2.0 * n * k + B * (2.0 * k + out * n)                                                    # noqa: E731
+    row = E * (8.0 * S + 8.0 + 2.0)                                # streams read and written, a result read and cleared, a normed row written
+    decode = {
+        "streams + norm": (2 * layers + 1) * B * row, "delta projections": nd * mul(n_d, E, 4.0), "recurrence set-up": nd * B * ch * 4.0 * (2 + 2 * 3),
+        "delta rule": nd * (B * (2.0 * state_d + 4.0 * n_d + 2.0 * Hd * Pd) + 2.0 * rank * Hd * (Dd + Pd)),
+        "recurrence projections": nl * mul(n_l, E, 4.0), "recurrence": nl * B * (2.0 * state_l + 4.0 * (2 * Hl * Dl + 2 * Hl * Pl)),
+        "gated norm": nl * B * Hl * Pl * 10.0, "qkv product": na * mul(n_qkv, E, 4.0), "query product": nq * mul(n_q, E, 4.0),
+        "rotary + append": (na * n_qkv + nq * n_q) * B * 6.0,
+        "attention": (na + nq) * B * (seen_decode * G * (2 * D + DV) * 2.0 + 2.0 * H * (2 * D + DV)),
+        "output product": nd * mul(E, Hd * Pd, 8.0) + nl * mul(E, Hl * Pl, 8.0) + (na + nq) * mul(E, H * DV, 8.0),
+        "up product": layers * mul(F, E, 2.0), "down product": layers * mul(E, F, 8.0), "head product": mul(V, E, 4.0),
+    }
+    prefill = {
+        "streams + norm": ("bytes", 2 * layers * T * row), "delta projections": ("flops", nd * 2.0 * T * n_d * E), "recurrence set-up": ("bytes", nd * T * ch * 8.0),
+        "low-rank split": ("bytes", nd * T * 2 * rank * 8.0), "low-rank product": ("bytes", nd * T * Hd * (Dd + Pd) * 4.0),
+        # a step of the recurrence: decay, two sums over the state and its update, 7 operations a state element
+        "delta rule": ("flops32", nd * T * Hd * Dd * Pd * 7.0), "recurrence projections": ("flops", nl * 2.0 * T * n_l * E),
+        "recurrence": ("flops32", nl * T * 4.0 * Hl * Dl * Pl), "gated norm": ("bytes", (nl * Hl * Pl + nd * Hd * Pd) * T * 10.0),
+        "qkv product": ("flops", na * 2.0 * T * n_qkv * E), "query product": ("flops", nq * 2.0 * T * n_q * E), "rotary + append": ("bytes", (na * n_qkv + nq * n_q) * T * 6.0),
+        "attention": ("flops", (na + nq) * 2.0 * H * 2 * (D + DV) * seen_prefill),
+        "output product": ("flops", 2.0 * T * E * (nd * Hd * Pd + nl * Hl * Pl + (na + nq) * H * DV)),
+        "up product": ("flops", layers * 2.0 * T * E * F), "down product": ("flops", layers * 2.0 * T * E * F),
+    }
+    return {"decode": decode, "prefill": prefill}
+
+
+def bench_duratar(pk, rng, size="wide", layers=4, batch=8, prompt=PROMPT, steps=32, warmup=4) -> dict:
+    """Prompt and decode throughput of a Duratar model of ``layers`` layers at sizes that resemble a real model's layers (random weights),
+    beside a Fegidra model, the closest of the other designs (delta-rule and masked attention layers in turn, dense feed-forwards without a
+    gate), of the same width, projections, feed-forward, vocabulary and depth; every kernel class of both against its own bytes or operations."""
+    c = DURATAR_SIZES[size]
+    f = dict(width=c["width"], heads=c["heads"], kv_heads=c["kv_heads"], dim=2 * c["dim"], vdim=c["vdim"], chunk=c["window"], delta_heads=c["delta_heads"],
+             delta_dim=c["delta_dim"], rank=c["rank"], ff=c["ff"], vocab=c["vocab"])
+    configs = {"duratar": duratar_config(layers=layers, **c), "fegidra": fegidra_config(layers=layers, **f)}
+    out = {"size": size, "sizes": c, "beside": f, "layers": layers, "batch": batch, "prompt": prompt,
+           "between": "weights of a step exceed the L2", "peaks": pk, "fp32_cuda_core_tflops_nominal": round(FP32_TFLOPS, 1)}
+
+    def costs_of(name, cfg):
+        return duratar_costs(c, layers, batch, prompt + 2, prompt) if name == "duratar" else fegidra_costs(f, layers, batch, prompt + 2, prompt)
+
+    return _bench_models(configs, costs_of, c["vocab"], out, pk, rng, FP32_TFLOPS, batch, prompt, steps, warmup)
+
+
 def run_ours(args) -> dict:
     import numpy as np
     import torch
@@ -1083,9 +1168,9 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 and 64 and the two other shapes")
     ap.add_argument("--no-breakdown", action="store_true", help="skip the per-class timing of one decode and one prompt step")
-    ap.add_argument("--point", default="", choices=["", "long", "13b", "3b", "tiny", "fegidra", "pozirax", "fudelorn", "logirax"],
+    ap.add_argument("--point", default="", choices=["", "long", "13b", "3b", "tiny", "fegidra", "pozirax", "fudelorn", "logirax", "duratar"],
                     help="run one of the further workloads alone and print its figures (not the default run's one JSON line)")
-    ap.add_argument("--size", default="wide", choices=sorted(FEGIDRA_SIZES), help="with --point fegidra, pozirax, fudelorn or logirax: which sizes")
+    ap.add_argument("--size", default="wide", choices=sorted(FEGIDRA_SIZES), help="with --point fegidra, pozirax, fudelorn, logirax or duratar: which sizes")
     args = ap.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable": "the reference is a Rust workspace (no setup.py or pyproject) "
@@ -1105,7 +1190,8 @@ def main() -> int:
                "fegidra": lambda: bench_fegidra(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
                "pozirax": lambda: bench_pozirax(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
                "fudelorn": lambda: bench_fudelorn(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
-               "logirax": lambda: bench_logirax(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup)}[args.point]
+               "logirax": lambda: bench_logirax(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
+               "duratar": lambda: bench_duratar(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup)}[args.point]
         print(json.dumps({"point": args.point, **one()}))
         return 0
     print(json.dumps(run_ours(args)))

@@ -181,7 +181,7 @@ template <int D> __device__ __forceinline__ int da_offset(int r, int c) {
 // rows each.  With `scratch` the block takes one of gridDim.z / seqs shares of the pages and leaves its rows' parts there:
 // [row][H][split][2][DV + 2] floats, products then maximum (base 2) then sum.
 template <int DP, int VP, int WM, int STAGES>
-__global__ void __launch_bounds__(64 * WM)
+__global__ void __launch_bounds__(64 * WM, WM == 1 ? 1 : VP <= 128 ? 3 : 2)
 diff_tiles_kernel(const bf16* q, const bf16* k_cache, const bf16* v_cache, const int* __restrict__ page_table, const int* __restrict__ seq_rows,
                   const int* __restrict__ seq_slot, const int* __restrict__ seq_start, bf16* __restrict__ out, float* __restrict__ scratch, int splits, int H,
                   int G, int D, int DV, int max_pages, int n_pages, int window, int keep, float scale_log2, float lambda, float eps, float factor) {
@@ -309,10 +309,7 @@ diff_tiles_kernel(const bf16* q, const bf16* k_cache, const bf16* v_cache, const
 #pragma unroll
             for (int nb = 0; nb < 8; nb++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    s[nb][e] *= scale_log2;
-                    tmax[e >> 1] = fmaxf(tmax[e >> 1], s[nb][e]);
-                }
+                for (int e = 0; e < 4; e++) tmax[e >> 1] = fmaxf(tmax[e >> 1], s[nb][e]);
         } else {
 #pragma unroll
             for (int nb = 0; nb < 8; nb++)
@@ -320,7 +317,7 @@ diff_tiles_kernel(const bf16* q, const bf16* k_cache, const bf16* v_cache, const
                 for (int e = 0; e < 4; e++) {
                     const int i = e >> 1, t = p0 + nb * 8 + 2 * tq + (e & 1);
                     const bool seen = live[i] && t <= pos[i] && (t >= lo[i] || t < keep);
-                    s[nb][e] = seen ? s[nb][e] * scale_log2 : -INFINITY;
+                    s[nb][e] = seen ? s[nb][e] : -INFINITY;
                     tmax[i] = fmaxf(tmax[i], s[nb][e]);
                 }
         }
@@ -329,7 +326,7 @@ diff_tiles_kernel(const bf16* q, const bf16* k_cache, const bf16* v_cache, const
         for (int i = 0; i < 2; i++) {
             tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
             tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
-            const float mn = fmaxf(m[i], tmax[i]);
+            const float mn = fmaxf(m[i], tmax[i] * scale_log2);        // the scale is positive: the largest score is the largest product
             corr[i] = mn == -INFINITY ? 1.0f : fast_exp2(m[i] - mn);
             base[i] = mn == -INFINITY ? 0.0f : mn;
             m[i] = mn;
@@ -339,14 +336,16 @@ diff_tiles_kernel(const bf16* q, const bf16* k_cache, const bf16* v_cache, const
         for (int nb = 0; nb < 8; nb++)
 #pragma unroll
             for (int e = 0; e < 4; e++) {
-                s[nb][e] = fast_exp2(s[nb][e] - base[e >> 1]);
+                s[nb][e] = fast_exp2(fmaf(s[nb][e], scale_log2, -base[e >> 1]));
                 psum[e >> 1] += s[nb][e];
             }
         l[0] = l[0] * corr[0] + psum[0];
         l[1] = l[1] * corr[1] + psum[1];
+        if (__any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f)) {      // most pages raise no row's maximum
 #pragma unroll
-        for (int nd = 0; nd < ND; nd++) {
-            o[nd][0] *= corr[0]; o[nd][1] *= corr[0]; o[nd][2] *= corr[1]; o[nd][3] *= corr[1];
+            for (int nd = 0; nd < ND; nd++) {
+                o[nd][0] *= corr[0]; o[nd][1] *= corr[0]; o[nd][2] *= corr[1]; o[nd][3] *= corr[1];
+            }
         }
 #pragma unroll
         for (int kk = 0; kk < 4; kk++) {
@@ -498,9 +497,9 @@ static int tiles_launch(const void* q, const void* k_cache, const void* v_cache,
 }
 
 // Whether the tile kernel takes the sizes (else the rows kernel serves): widths multiples of 8, maps up to 128, values up to 256, at
-// most 64 heads a kv head.
+// most 32 heads a kv head.
 extern "C" int bc_diff_tiles_accepts(int H, int G, int D, int DV) {
-    return G > 0 && H % G == 0 && H / G <= 64 && D % 8 == 0 && D > 0 && D <= 128 && DV % 8 == 0 && DV > 0 && DV <= 256;
+    return G > 0 && H % G == 0 && H / G <= 32 && D % 8 == 0 && D > 0 && D <= 128 && DV % 8 == 0 && DV > 0 && DV <= 256;
 }
 
 // q: [rows, H, 2, D] bf16; out: [rows, H, DV]; sequence s owns rows seq_rows[s] .. seq_rows[s + 1], lives in slot seq_slot[s] (negative:
@@ -513,6 +512,7 @@ extern "C" int bc_diff_tiles_bf16(const void* q, const void* k_cache, const void
     BC_CHECK_ARG(bc_diff_tiles_accepts(H, G, D, DV), "diff_tiles: H=%d G=%d D=%d DV=%d is outside what this kernel takes", H, G, D, DV);
     BC_CHECK_ARG(seqs >= 0 && splits >= 1 && (long long)seqs * splits <= 65535 && max_new >= 0 && max_new < 65535, "diff_tiles: bad sizes seqs=%d splits=%d max_new=%d",
                  seqs, splits, max_new);
+    BC_CHECK_ARG(scale > 0.0f, "diff_tiles: a scale of %g is not positive", (double)scale);
     BC_CHECK_ARG(window >= 0 && keep >= 0 && (splits == 1 || (scratch && row_slot)), "diff_tiles: bad window %d, kept %d or no scratch", window, keep);
     BC_CHECK_ARG((uintptr_t)q % 4 == 0 && (uintptr_t)out % 4 == 0 && (uintptr_t)k_cache % 16 == 0 && (uintptr_t)v_cache % 16 == 0, "diff_tiles: unaligned operands");
     if (seqs == 0 || max_new == 0) return BC_OK;
@@ -524,7 +524,7 @@ extern "C" int bc_diff_tiles_bf16(const void* q, const void* k_cache, const void
 #define DA_V(DP_, VP_)                    \
     do {                                  \
         if (few) DA_GO(DP_, VP_, 1);      \
-        else DA_GO(DP_, VP_, 4);          \
+        else DA_GO(DP_, VP_, 2);          \
     } while (0)
 #define DA_D(DP_)                         \
     do {                                  \

@@ -43,15 +43,17 @@ extern "C" int bc_sm_count() {
 // given, once a device, a word of mapped host memory as well: the first wait that gives up
 // writes its code there, and the host reads it after any synchronisation of its own (a copy
 // of token ids, say) at no cost.  Word 0: the tensor-core product; word 1: the tcgen05
-// prompt attention.
+// prompt attention; word 2: the decode attention; word 3: the tcgen05 differential attention.
 extern "C" int bc_gemm_tc_bind_host_word(int*);
 extern "C" int bc_attention_prefill_tc_bind_host_word(int*);
 extern "C" int bc_attention_decode_bind_host_word(int*);
+extern "C" int bc_diff_attention_tc_bind_host_word(int*);
 extern "C" int bc_gemm_tc_status(int);
 extern "C" int bc_attention_prefill_tc_status(int);
 extern "C" int bc_attention_decode_status(int);
+extern "C" int bc_diff_attention_tc_status(int);
 
-#define BC_STATUS_UNITS 3
+#define BC_STATUS_UNITS 4
 static int* g_status_words[64];   // per device: BC_STATUS_UNITS ints of mapped host memory
 
 extern "C" int bc_status_bind() {
@@ -73,6 +75,7 @@ extern "C" int bc_status_bind() {
     int st = bc_gemm_tc_bind_host_word(seen_by_device + 0);
     if (st == 0) st = bc_attention_prefill_tc_bind_host_word(seen_by_device + 1);
     if (st == 0) st = bc_attention_decode_bind_host_word(seen_by_device + 2);
+    if (st == 0) st = bc_diff_attention_tc_bind_host_word(seen_by_device + 3);
     if (st != 0) {
         bc_set_error("status_bind: cannot hand the status words to the kernels: %s", cudaGetErrorString((cudaError_t)st));
         return st;
@@ -92,7 +95,8 @@ extern "C" int bc_status_peek(int unit, int reset) {
         g_status_words[dev][unit] = 0;
         if (unit == 0) bc_gemm_tc_status(1);
         else if (unit == 1) bc_attention_prefill_tc_status(1);
-        else bc_attention_decode_status(1);
+        else if (unit == 2) bc_attention_decode_status(1);
+        else bc_diff_attention_tc_status(1);
     }
     return v;
 }

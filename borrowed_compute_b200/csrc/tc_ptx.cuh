@@ -15,7 +15,11 @@ enum { EPI_STORE = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3, EPI_RE
 // float; the store rounds once); EPI_XIELU is a v^2 + v/2 above zero and b (e^v - 1 - v) + v/2 below; EPI_SILU_F32 gates output columns
 // n < cols by their own sigmoid and stores floats; the others leave it.
 template <int EPI> __device__ __forceinline__ float epi_plain(float v, float a = 0.0f, float b = 0.0f, int n = 0, int cols = 0) {
-    if (EPI == EPI_XIELU) return fmaf(0.5f, v, v > 0.0f ? a * v * v : b * (__expf(v) - 1.0f - v));
+    if (EPI == EPI_XIELU) {
+        // Both halves of v, each zero where the other holds, so that there is nothing to branch on.
+        const float t = fmaxf(v, 0.0f), n = fminf(v, 0.0f);
+        return fmaf(fmaf(a, t, 0.5f), t, fmaf(b, __expf(n), fmaf(0.5f - b, n, -b)));
+    }
     if (EPI == EPI_SILU_F32) return n < cols ? __fdividef(v, 1.0f + __expf(-v)) : v;
     if (EPI == EPI_RELU2) {
         v = fmaxf(v, 0.0f);

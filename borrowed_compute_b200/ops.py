@@ -437,7 +437,7 @@ def gemm_tc_status(reset: bool = True) -> int:
 def set_wait_cycles(cycles: int = 0) -> None:
     """The most clocks a bounded wait inside the tensor-core kernels may take before it gives
     up and records its status (0: back to the default, about a second)."""
-    for unit in ("gemm_tc", "attention_prefill_tc", "attention_decode"):
+    for unit in ("gemm_tc", "attention_prefill_tc", "attention_decode", "diff_attention_tc"):
         st = _fn(f"bc_{unit}_set_wait_cycles")(ctypes.c_longlong(int(cycles)))
         if st != 0:
             raise KernelError(f"setting the wait limit of {unit} failed ({st})")
@@ -451,7 +451,8 @@ def gemm_tc_test_starve_next_launch() -> None:
 
 # ------------------------------------------------------------ errors that reach the caller
 
-_STATUS_UNITS = ("the tensor-core product (gemm_tc)", "the tcgen05 prompt attention (attention_prefill_tc)", "the decode attention (attention_decode)")
+_STATUS_UNITS = ("the tensor-core product (gemm_tc)", "the tcgen05 prompt attention (attention_prefill_tc)", "the decode attention (attention_decode)",
+                 "the tcgen05 differential attention (diff_attention_tc)")
 _WAITS = {
     0: {1: "the loader's wait for a free stage", 2: "the wait for a stage's operands", 3: "the epilogue's wait for the accumulator",
         4: "the wait for the epilogue to hand the accumulator back"},
@@ -459,6 +460,9 @@ _WAITS = {
         5: "the wait for a page", 6: "the softmax's wait for scores", 7: "the wait for a product that frees P", 8: "the wait for the last product",
         9: "the wait before a rescale"},
     2: {1: "the wait for a page of keys and values"},
+    3: {1: "the loader's wait for a free stage", 2: "the wait for the queries", 3: "the wait for the first pages", 4: "the wait for P",
+        5: "the wait for a page", 6: "the softmax's wait for scores", 7: "the wait for a product that frees P", 8: "the wait for the last product",
+        9: "the wait before a rescale"},
 }
 _bound_devices = set()
 
@@ -1111,6 +1115,30 @@ def diff_rows(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, pag
 def diff_tiles_accepts(heads: int, kv_heads: int, head_dim: int, value_dim: int, dtype: torch.dtype) -> bool:
     """Whether the tensor-core tile kernel takes these sizes (bf16, widths multiples of 8: maps up to 128, values up to 256)."""
     return dtype == torch.bfloat16 and bool(_fn("bc_diff_tiles_accepts")(_c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim)))
+
+
+def diff_attention_tc_accepts(heads: int, kv_heads: int, head_dim: int, value_dim: int, dtype: torch.dtype) -> bool:
+    """Whether the tcgen05 kernel for prompts takes these sizes (bf16, maps of 64 or 128, values of 64 or 128)."""
+    return dtype == torch.bfloat16 and bool(_fn("bc_diff_attention_tc_accepts")(_c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim)))
+
+
+def diff_attention_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor, seq_rows: torch.Tensor, seq_slot: torch.Tensor,
+                      seq_start: torch.Tensor, out: torch.Tensor, seqs: int, max_new: int, heads: int, kv_heads: int, head_dim: int, value_dim: int, window: int,
+                      keep_first: int, scale: float, lam: float, eps: float, factor: float) -> None:
+    """What diff_tiles computes, for prompts on the tcgen05 tensor cores: scores and both maps' outputs in tensor memory."""
+    _diff_check("diff_attention_tc", q, k_cache, v_cache, page_table, out, heads, kv_heads, head_dim, value_dim)
+    _need(q, "q", torch.bfloat16)
+    for t, name in ((seq_rows, "seq_rows"), (seq_slot, "seq_slot"), (seq_start, "seq_start")):
+        _need(t, name, torch.int32)
+    if seq_rows.numel() < seqs + 1 or seq_slot.numel() < seqs or seq_start.numel() < seqs:
+        raise KernelError("diff_attention_tc: fewer sequence entries than sequences")
+    _bounds("diff_attention_tc: seq_slot", seq_slot, page_table.shape[0], seqs, lowest=-1)
+    _bounds("diff_attention_tc: seq_rows", seq_rows, q.shape[0] + 1, seqs + 1)
+    _bounds("diff_attention_tc: page_table", page_table, k_cache.shape[0], lowest=-1)
+    _call(_fn("bc_diff_attention_tc_bf16"), _ptr(q), _c_int(q.shape[0]), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(seq_rows), _ptr(seq_slot),
+          _ptr(seq_start), _ptr(out), _c_int(seqs), _c_int(max_new), _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim),
+          _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_int(keep_first), _c_float(scale), _c_float(lam), _c_float(eps),
+          _c_float(factor), _stream())
 
 
 def diff_tiles_splits(seqs: int, kv_heads: int, reach: int, window: int, keep_first: int) -> int:

@@ -27,7 +27,9 @@ from .. import ops
 from . import products
 from .base import MIXERS, POSITION_ENCODINGS, CacheNeed, Mixer, RunMemory, Runtime, StepContext, TensorSpec
 
-force_rows = False      # tests: take the one-warp-a-row kernel (the checked twin) for bfloat16 too
+# Tests: "rows" (the one-warp-a-row kernel, the checked twin), "tiles" (mma.sync tiles) or "tc" (tcgen05) wherever the sizes allow it;
+# None: the part chooses.
+force: Optional[str] = None
 force_splits = 0        # tests: share a row's pages out over this many blocks in steps of few rows (0: the part chooses)
 
 
@@ -73,6 +75,14 @@ class DifferentialAttention(Mixer):
         self.lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + self.diff)      # of the weights alone: once
         self.position.load({}, rt)
 
+    def path(self, ctx: StepContext, dtype: torch.dtype) -> str:
+        """Which kernel this step's rows take: prompts tcgen05 tiles where the widths are 64 or 128, other widths and steps of few rows a
+        sequence mma.sync tiles, the 32-bit path and what no tile takes one warp a row."""
+        H, G, D, DV = self.heads, self.kv_heads, self.head_dim, self.value_dim
+        if force in (None, "tc") and not ctx.decode and ctx.max_new * (H // G) > 16 and ops.diff_attention_tc_accepts(H, G, D, DV, dtype):
+            return "tc"
+        return "tiles" if force != "rows" and ops.diff_tiles_accepts(H, G, D, DV, dtype) else "rows"
+
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx: StepContext, mem: RunMemory) -> None:
         if len(mem.planes) != 2:
             raise RuntimeError("differential attention was given no cache: the cache does not serve this run")
@@ -87,8 +97,12 @@ class DifferentialAttention(Mixer):
                               write_cache=mem.writes and self.own_kv, value_heads=G if self.own_kv else 0)
         att = torch.empty((rows, H * DV), dtype=x.dtype, device=x.device)
         numbers = dict(window=self.window, keep_first=self.keep_first, scale=self.scale, lam=self.lam, eps=self.norm_eps, factor=1.0 - self.diff)
-        if force_rows or not ops.diff_tiles_accepts(H, G, D, DV, x.dtype):
+        path = self.path(ctx, x.dtype)
+        if path == "rows":
             ops.diff_rows(q, mem.k_pages, mem.v_pages, mem.page_table, ctx.row_pos, ctx.row_slot, att, H, G, D, DV, **numbers)
+        elif path == "tc":
+            ops.diff_attention_tc(q, mem.k_pages, mem.v_pages, mem.page_table, ctx.seq_rows, ctx.seq_slot, ctx.seq_start, att, ctx.seqs, ctx.max_new, H, G, D, DV,
+                                  **numbers)
         else:
             splits = 1
             if ctx.decode:
