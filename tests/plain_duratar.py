@@ -256,3 +256,157 @@ def generate(cfg, tensors, prompt, n):
     for _ in range(n):
         ids.append(int(np.argmax(logits(cfg, tensors, ids)[-1])))
     return ids[len(prompt):]
+
+
+# ------------------------------------------------------------------------- small models and their weights
+
+def to_bf16(a):
+    """float32 values rounded to the nearest bfloat16 (ties to even)."""
+    bits = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32).astype(np.uint64)
+    bits = (bits + 0x7FFF + ((bits >> 16) & 1)) & 0xFFFF0000
+    return bits.astype(np.uint32).view(np.float32).reshape(np.shape(a))
+
+
+def attention_mixer(heads, kv_heads, dim, vdim, window=0, keep=0, rot=0, base=10000.0, scaling=None, scale=None, diff=0.5, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": 1.5 / dim ** 0.5 if scale is None else scale, "diff": diff}
+    if window:
+        m["mask"] = {"size": window, "keep_first": keep}
+    if rot:
+        m["rot"] = {"dims": rot, "base": base}
+        if scaling:
+            m["rot"]["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return m
+
+
+def lightning_mixer(heads, dim, vdim, slowest=0.99):
+    return {"heads": heads, "dim": dim, "vdim": vdim, "decay": [float(d) for d in np.linspace(0.5, slowest, heads)]}
+
+
+def delta_mixer(heads, kv_heads, dim, vdim, conv, decay_rank, gate_rank):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv, "decay_rank": decay_rank, "gate_rank": gate_rank}
+
+
+def model(vocab, width, streams, layers, eps=1e-5):
+    """``layers``: (mixer, ff) pairs; the mixer's keys tell its type, ff 0 leaves the feed-forward out."""
+    kind = lambda m: "lightning" if "decay" in m else "channel_delta" if "conv" in m else "attention"          # noqa: E731
+    return {"architecture": "Duratar", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps},
+            "layers": [{"type": kind(m), "mixer": m, "mlp": {"kind": "dense", "ff": f} if f else None} for m, f in layers]}
+
+
+SMALL = {
+    # three streams; shared keys under a wider window than their owner's; shared delta keys; a layer without a feed-forward
+    "A": model(131, 72, 3, [
+        (attention_mixer(4, 2, 16, 24, 24, 3, 8, 500.0, (3.0, 1.0, 4.0, 60)), 40),
+        (delta_mixer(4, 2, 12, 20, 4, 8, 16), 56),
+        (attention_mixer(4, 2, 16, 24, 50, 5, 8, 500.0, (3.0, 1.0, 4.0, 60), diff=0.3, kv_from=0), 0),
+        (lightning_mixer(3, 16, 12), 40)]),
+    # one stream, one head, no mask, no rotation, a convolution of one tap, widths that nothing divides
+    "B": model(97, 50, 1, [
+        (lightning_mixer(2, 10, 14), 22),
+        (attention_mixer(3, 1, 10, 6, diff=0.2), 30),
+        (delta_mixer(3, 1, 18, 10, 1, 5, 3), 0),
+        (attention_mixer(3, 1, 10, 6, 70, 66, diff=0.7, kv_from=1), 26),
+        (delta_mixer(1, 1, 6, 7, 2, 4, 8), 22)], eps=1e-6),
+    # widths the tensor-core kernels take
+    "C": model(200, 128, 2, [
+        (attention_mixer(4, 2, 64, 128, 100, 66, 32, 10000.0), 96),
+        (attention_mixer(4, 2, 64, 128, 0, 0, 32, 10000.0, kv_from=0), 64),
+        (delta_mixer(2, 2, 64, 64, 3, 16, 24), 96),
+        (attention_mixer(2, 1, 48, 40, 65, 2, 48, 300.0), 64),
+        (lightning_mixer(2, 128, 64, 0.995), 96)]),
+}
+
+
+def tensor_shapes(cfg):
+    E, S, V = cfg["width"], cfg["streams"], cfg["vocab"]
+    out = {"embed": (V, E), "embed.norm": (), "final.norm": (), "head": (V, E)}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        x = p + "mix."
+        for n in ("1", "2") if L.get("mlp") else ("1",):
+            out.update({p + "norm" + n: (), p + "ls" + n: (E,), p + f"hc{n}.in": (S,), p + f"hc{n}.out": (S,), p + f"hc{n}.mix": (S, S)})
+        H, d, v = m["heads"], m["dim"], m["vdim"]
+        out[x + "o"] = (E, H * v)
+        if L["type"] == "attention":
+            out.update({x + "q": (2 * H * d, E), x + "q.norm": (d,), **{x + n: (d,) for n in ("lq1", "lk1", "lq2", "lk2")}})
+            if m.get("kv_from") is None:
+                G = m["kv_heads"]
+                out.update({x + "k": (2 * G * d, E), x + "k.norm": (d,), x + "v": (G * v, E)})
+        elif L["type"] == "lightning":
+            out.update({x + "q": (H * d, E), x + "k": (H * d, E), x + "v": (H * v, E), x + "g": (H * v, E), x + "norm": (H * v,)})
+        else:
+            G, taps = m["kv_heads"], m["conv"]
+            out.update({x + "q": (G * d, E), x + "k": (G * d, E), x + "v": (H * v, E), x + "q.conv": (G * d, taps), x + "k.conv": (G * d, taps),
+                        x + "v.conv": (H * v, taps), x + "b": (H, E), x + "A_log": (H,), x + "norm": (v,), x + "dt_bias": (H * d,),
+                        x + "a1": (m["decay_rank"], E), x + "a2": (H * d, m["decay_rank"]), x + "g1": (m["gate_rank"], E), x + "g2": (H * v, m["gate_rank"])})
+        if L.get("mlp"):
+            f = L["mlp"]["ff"]
+            out.update({p + "mlp.up": (f, E), p + "mlp.down": (E, f), p + "mlp.act": (2,)})
+    return out
+
+
+def make_weights(cfg, seed):
+    """Random weights that bfloat16 holds exactly: matrices of spread 1 / sqrt(inputs), norm numbers around one, connections that mix the
+    streams well, channels of the delta rule that forget within a few to a few hundred tokens."""
+    rng, t = np.random.default_rng(seed), {}
+    S = cfg["streams"]
+    for name, shape in tensor_shapes(cfg).items():
+        last = name.split(".")[-1]
+        if "norm" in name:
+            a = 1.0 + 0.3 * rng.uniform(-1, 1, shape)
+        elif last in ("ls1", "ls2"):
+            a = rng.uniform(0.4, 1.2, shape)
+        elif last == "in":
+            a = rng.uniform(0.3, 1.4, shape) / S
+        elif last == "out":
+            a = rng.uniform(0.5, 1.2, shape)
+        elif last == "mix":
+            a = 0.75 * np.eye(S) + 0.25 * rng.standard_normal((S, S)) / math.sqrt(S)
+        elif last in ("lq1", "lk1", "lq2", "lk2"):
+            a = 0.5 * rng.standard_normal(shape) / shape[0] ** 0.25
+        elif last == "A_log":
+            a = rng.uniform(-2.0, 1.0, shape)
+        elif last == "dt_bias":
+            a = rng.uniform(-5.0, -1.0, shape)
+        elif last == "act":
+            a = rng.uniform(-1.5, 1.5, shape)
+        elif last == "conv":
+            a = rng.uniform(-0.6, 0.6, shape)
+            a[:, -1] += 0.8
+        elif name == "embed":
+            a = rng.standard_normal(shape)
+        else:
+            a = rng.standard_normal(shape) / math.sqrt(shape[-1]) * (2.0 if last in ("head", "g", "g2", "a2", "b") else 1.0)
+        t[name] = to_bf16(a)
+    return t
+
+
+def draw_config(rng):
+    """A configuration whose sizes, constants and order of layers are drawn."""
+    E, layers, owners = int(rng.choice([24, 40, 56, 64, 72, 128])), [], []
+    for i in range(int(rng.integers(2, 6))):
+        u = rng.random()
+        if u < 0.45:
+            if owners and rng.random() < 0.5:
+                j = int(rng.choice(owners))
+                m = dict(layers[j][0], kv_from=j, diff=float(rng.choice([0.1, 0.8])))
+                m.pop("mask", None)
+                if rng.random() < 0.8:
+                    m["mask"] = {"size": int(rng.choice([1, 7, 64, 90])), "keep_first": int(rng.choice([0, 2, 65]))}
+            else:
+                G, d = int(rng.choice([1, 2, 3])), int(rng.choice([8, 10, 16, 40, 48, 64, 128]))
+                scaling = (float(rng.choice([2.0, 8.0])), 1.0, float(rng.choice([2.0, 4.0])), int(rng.choice([32, 64, 300]))) if rng.random() < 0.6 else None
+                m = attention_mixer(G * int(rng.choice([1, 2, 3, 5])), G, d, int(rng.choice([6, 8, 24, 64, 104, 128])), int(rng.choice([0, 1, 5, 33, 64, 100])),
+                                    int(rng.choice([0, 1, 4, 64, 66])), int(rng.choice([0, d // 2 // 2 * 2, d])), float(rng.choice([100.0, 10000.0])), scaling,
+                                    diff=float(rng.choice([0.2, 0.5, 0.8])))
+                owners.append(i)
+        elif u < 0.7:
+            m = lightning_mixer(int(rng.choice([1, 2, 5])), int(rng.choice([6, 8, 16, 40, 130])), int(rng.choice([4, 12, 33, 64])), float(rng.choice([0.9, 0.999])))
+        else:
+            G = int(rng.choice([1, 2]))
+            m = delta_mixer(G * int(rng.choice([1, 2, 3])), G, int(rng.choice([6, 8, 16, 20, 64, 100])), int(rng.choice([5, 8, 32, 72])), int(rng.choice([1, 2, 3, 4, 6])),
+                            int(rng.choice([3, 8, 24])), int(rng.choice([4, 16, 20])))
+        layers.append((m, int(rng.choice([0, 8, 20, 48]))))
+    return model(int(rng.choice([50, 131, 200])), E, int(rng.choice([1, 2, 4, 5, 9])), layers, eps=float(rng.choice([1e-6, 1e-5, 1e-3])))

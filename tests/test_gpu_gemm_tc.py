@@ -30,6 +30,15 @@ def f64(t):
     return t.detach().float().cpu().numpy().astype(np.float64)
 
 
+def xielu(z, a, b):
+    low = np.minimum(z, 0.0)
+    return np.where(z > 0, a * z * z, b * (np.expm1(low) - low)) + 0.5 * z
+
+
+def silu_below(z, cols):
+    return np.where(np.arange(z.shape[1]) < cols, z / (1.0 + np.exp(-z)), z)
+
+
 @pytest.mark.parametrize("T,N,K,splits", SHAPES)
 def test_gemm_tc_all_epilogues(T, N, K, splits):
     from borrowed_compute_b200 import ops
@@ -63,6 +72,14 @@ def test_gemm_tc_all_epilogues(T, N, K, splits):
     out16.fill_(7.0)
     ops.gemm_tc(x, wn, out16, ops.EPI_RELU2, splits=splits)
     assert np.abs(f64(out16) - squared).max() <= 2.0 ** -8 * (1 + np.abs(squared).max()), "the square of relu"
+    curve, partly = xielu(full[:, :N], 0.7, 1.3), silu_below(full[:, :N], N // 3)
+    out16.fill_(7.0)
+    ops.gemm_tc(x, wn, out16, ops.EPI_XIELU, splits=splits, act=(0.7, 1.3))
+    assert np.abs(f64(out16) - curve).max() <= 2.0 ** -8 * (1 + np.abs(curve).max()), "xIELU"
+    ops.gemm_tc(x, wn, out32, ops.EPI_SILU_F32, splits=splits, cols=N // 3)
+    assert np.abs(f64(out32) - partly).max() <= 2e-5 * scale, "silu of the first columns"
+    with pytest.raises(ops.KernelError, match="EPI_XIELU"):
+        ops.gemm_tc(x, wn, out16, ops.EPI_XIELU, splits=splits)
     assert ops.gemm_tc_status() == 0
 
 
@@ -87,11 +104,15 @@ def test_gemm_tc_splits_agree_through_cluster_and_through_scratch(T, N, K, split
             ops.gemm_tc(x, wn, acc, ops.EPI_ADD_F32, splits=splits)
             act = torch.full((T, N), 7.0, dtype=torch.bfloat16, device="cuda")
             ops.gemm_tc(x, w, act, ops.EPI_SWIGLU, splits=splits)
-            results.append((out32, out16, acc, act))
+            curve = torch.full((T, N), 7.0, dtype=torch.bfloat16, device="cuda")
+            ops.gemm_tc(x, wn, curve, ops.EPI_XIELU, splits=splits, act=(0.4, 2.0))
+            partly = torch.full((T, N), 7.0, dtype=torch.float32, device="cuda")
+            ops.gemm_tc(x, wn, partly, ops.EPI_SILU_F32, splits=splits, cols=N - 5)
+            results.append((out32, out16, acc, act, curve, partly))
     finally:
         ops.set_gemm_tc_cluster(True)
     assert ops.gemm_tc_status() == 0
-    for a, b, name in zip(results[0], results[1], ("float store", "bf16 store", "residual add", "SwiGLU")):
+    for a, b, name in zip(results[0], results[1], ("float store", "bf16 store", "residual add", "SwiGLU", "xIELU", "silu of the first columns")):
         assert torch.equal(a, b), name
     full = f64(x) @ f64(wn).T
     assert np.abs(f64(results[0][0]) - full).max() <= 2e-5 * (1.0 + np.abs(full).max())
@@ -122,6 +143,10 @@ def test_gemm_tc_many_tokens_on_pairs_of_sms_and_on_single_blocks(T, N, K, paire
         ops.gemm_tc(x, w, act, ops.EPI_SWIGLU, splits=1)
         sq = torch.full((T, N), 7.0, dtype=torch.bfloat16, device="cuda")
         ops.gemm_tc(x, wn, sq, ops.EPI_RELU2, splits=1)
+        curve = torch.full((T, N), 7.0, dtype=torch.bfloat16, device="cuda")
+        ops.gemm_tc(x, wn, curve, ops.EPI_XIELU, splits=1, act=(1.5, 0.6))
+        partly = torch.full((T, N), 7.0, dtype=torch.float32, device="cuda")
+        ops.gemm_tc(x, wn, partly, ops.EPI_SILU_F32, splits=1, cols=N // 2)
     finally:
         ops.set_gemm_tc_pair(True)
         ops.set_gemm_tc_pair_tokens(0)
@@ -134,6 +159,9 @@ def test_gemm_tc_many_tokens_on_pairs_of_sms_and_on_single_blocks(T, N, K, paire
     assert np.abs(f64(act) - ref).max() <= 2.0 ** -8 * (1 + np.abs(ref).max()), "SwiGLU"
     squared = np.maximum(full[:, :N], 0.0) ** 2
     assert np.abs(f64(sq) - squared).max() <= 2.0 ** -8 * (1 + np.abs(squared).max()), "the square of relu"
+    want = xielu(full[:, :N], 1.5, 0.6)
+    assert np.abs(f64(curve) - want).max() <= 2.0 ** -8 * (1 + np.abs(want).max()), "xIELU"
+    assert np.abs(f64(partly) - silu_below(full[:, :N], N // 2)).max() <= 2e-5 * scale, "silu of the first columns"
 
 
 def test_gemm_tc_matches_the_cuda_core_twin():

@@ -111,6 +111,13 @@ def test_gemm_simt(dtype, M, N, K):
     squared = np.maximum(full[:, :N], 0.0) ** 2
     ops.gemm_simt(xd, wd[:N].contiguous(), out, ops.EPI_RELU2)
     assert np.abs(f64(out) - squared).max() <= out_tol(dtype, squared)
+    z = full[:, :N]
+    curve = np.where(z > 0, 0.7 * z * z, 1.3 * (np.expm1(np.minimum(z, 0.0)) - np.minimum(z, 0.0))) + 0.5 * z
+    ops.gemm_simt(xd, wd[:N].contiguous(), out, ops.EPI_XIELU, act=(0.7, 1.3))
+    assert np.abs(f64(out) - curve).max() <= out_tol(dtype, curve)
+    ops.gemm_simt(xd, wd[:N].contiguous(), out32, ops.EPI_SILU_F32, cols=N // 2)
+    partly = np.where(np.arange(N) < N // 2, z / (1 + np.exp(-z)), z)
+    assert np.abs(f64(out32) - partly).max() <= 1e-5 * (1 + np.abs(full).max())
 
 
 def poison(kp, vp, table, lengths, drop_before=None):
