@@ -50,15 +50,16 @@ template <int R> __device__ __forceinline__ void cd_load(const float* vec, int l
     }
 }
 template <int R> __device__ __forceinline__ void cd_load_column(const float* col, int lane, int D, bool ok, float* s) {
-    if (R >= 4 && D % 4 == 0) {
+    if constexpr (R >= 4) {
+        if (D % 4 == 0) {
 #pragma unroll
-        for (int q = 0; q < R; q += 4) {
-            const int i = cd_channel<R>(lane, q);
-            const float4 v = ok && i < D ? *reinterpret_cast<const float4*>(col + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            s[q] = v.x; s[q + 1 < R ? q + 1 : q] = v.y;
-            if (R >= 4) { s[q + 2 < R ? q + 2 : q] = v.z; s[q + 3 < R ? q + 3 : q] = v.w; }
+            for (int q = 0; q < R; q += 4) {
+                const int i = cd_channel<R>(lane, q);
+                const float4 v = ok && i < D ? *reinterpret_cast<const float4*>(col + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                s[q] = v.x; s[q + 1] = v.y; s[q + 2] = v.z; s[q + 3] = v.w;
+            }
+            return;
         }
-        return;
     }
 #pragma unroll
     for (int q = 0; q < R; q++) {

@@ -388,7 +388,7 @@ def test_one_key_that_matters_at_every_edge(dtype, path, which, window, keep, st
 
 @pytest.mark.parametrize("dtype,path", DIFF_PATHS)
 @pytest.mark.parametrize("H,G,D,DV,rot,window,keep", [(1, 1, 8, 8, 8, 0, 0), (6, 2, 40, 24, 20, 100, 5), (5, 1, 10, 6, 4, 50, 1), (3, 3, 128, 256, 64, 64, 64), (16, 4, 64, 128, 32, 77, 0),
-                                                      (4, 1, 48, 96, 24, 300, 7), (8, 8, 24, 40, 24, 31, 2), (40, 2, 64, 64, 0, 90, 33), (2, 2, 128, 128, 0, 0, 0),
+                                                      (5, 1, 48, 80, 16, 300, 7), (8, 8, 24, 40, 24, 31, 2), (40, 2, 64, 64, 0, 90, 33), (2, 2, 128, 128, 0, 0, 0),
                                                       (4, 2, 128, 64, 128, 65, 3), (3, 1, 64, 200, 0, 128, 70)])
 def test_differential_attention_in_other_sizes(dtype, path, H, G, D, DV, rot, window, keep):
     """One head; groups of many heads; widths that are no power of two, values wider and narrower than a map; everything turning, or nothing;
