@@ -60,7 +60,7 @@ class PagedCache:
         self.n_pages = n_pages
         self.slots = SlotTable(n_slots, n_pages, max_seq, [GroupPlan(g.need.window, g.need.chunk, g.need.keep_first) for g in self.groups])
         for g in self.groups:
-            g.planes = [torch.zeros((len(g.runs), n_pages, heads, PAGE, width), dtype=rt.dtype, device=rt.device)
+            g.planes = [torch.zeros((len(g.runs), n_pages, heads, PAGE, width), dtype=g.need.dtype or rt.dtype, device=rt.device)
                         for heads, width in g.need.planes]
             g.host_table = torch.full((n_slots, self.slots.max_pages), -1, dtype=torch.int32).pin_memory() \
                 if rt.device.type == "cuda" else torch.full((n_slots, self.slots.max_pages), -1, dtype=torch.int32)

@@ -56,14 +56,14 @@ extern "C" int bc_attention_decode_set_trace(long long* buf) { return (int)cudaM
 // The four computing warps among themselves (the fifth warp, where there is one, is not part of it).
 __device__ __forceinline__ void ad_workers_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-template <int D, bool TMA>
+template <int D, bool TMA, bool BIAS>
 __global__ void __launch_bounds__(TMA ? AD_THREADS_TMA : AD_THREADS)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
                         const int* __restrict__ page_table, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                         bf16* __restrict__ out, float* __restrict__ scratch, int* __restrict__ counters, int H, int G, int max_pages,
                         int n_pages, int window, float scale_log2, const float2* __restrict__ cos_sin, int pairing, int fuse,
                         int k_off, int v_off, bf16* __restrict__ k_write, bf16* __restrict__ v_write, int use_cluster, int sink,
-                        float out_scale) {
+                        float out_scale, const float* __restrict__ bias, int bias_reach) {
     constexpr int CHUNKS = D / 8;              // 16-byte chunks a row
     constexpr int TILE_BYTES = 64 * D * 2;     // one page of one kv head
     constexpr int KD = D / 16;                 // k-steps of Q K^T
@@ -252,9 +252,27 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     for (int i = 0; i < ND; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;   // rows gq and gq + 8
 
+    // Biases by distance (a table as in common.cuh, in log2 units; BIAS): this thread's two heads, and their numbers past the reach.
+    const float* kv_bias = BIAS ? bias_of_kv_head(bias, bias_reach, group, g) : nullptr;
+    const int head0 = gq < group ? gq : 0, head1 = gq + 8 < group ? gq + 8 : 0;
+    const float far0 = BIAS ? __ldg(kv_bias + (size_t)(bias_reach - 1) * group + head0) : 0.0f;
+    const float far1 = BIAS ? __ldg(kv_bias + (size_t)(bias_reach - 1) * group + head1) : 0.0f;
+
     bool waits_ok = true;
     for (int it = 0; it < n_tiles; it++) {
         AD_STAMP(16 + 6 * it);
+        float add[BIAS ? 2 : 1][4];      // this thread's positions of the page, asked for before the page is waited for
+        if (BIAS) {
+            const int first = (t_begin + it) * BC_PAGE + 16 * warp;
+            const bool far = pos - (first + 15) >= bias_reach - 1;
+#pragma unroll
+            for (int nb = 0; nb < 2; nb++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int n = min(max(pos - (first + nb * 8 + 2 * tq + (e & 1)), 0), bias_reach - 1);
+                    add[BIAS ? nb : 0][e] = far ? (e < 2 ? far0 : far1) : __ldg(kv_bias + (size_t)n * group + (e < 2 ? head0 : head1));
+                }
+        }
         if (TMA) {
             // Every thread sees the page arrive for itself; a warp goes on or gives up as one.  A
             // warp that has given up (its wait ran out: recorded) still walks through the pages
@@ -349,7 +367,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             for (int e = 0; e < 4; e++) {
                 const int t = tile * BC_PAGE + key0 + nb * 8 + 2 * tq + (e & 1);
                 const bool seen = page_ok && t >= lo && t <= pos;
-                s[nb][e] = seen ? s[nb][e] * scale_log2 : -INFINITY;
+                s[nb][e] = !seen ? -INFINITY : BIAS ? fmaf(s[nb][e], scale_log2, add[BIAS ? nb : 0][e]) : s[nb][e] * scale_log2;
                 if (e < 2) tmax0 = fmaxf(tmax0, s[nb][e]);
                 else tmax1 = fmaxf(tmax1, s[nb][e]);
             }
@@ -554,6 +572,8 @@ struct FusedRope {
     bool allow_cluster;     // splits may run as a thread-block cluster (else they go through scratch memory)
     int sink;               // 1: one added to the softmax's denominator (a position of score 0 without a value)
     float out_scale;        // a factor on the result
+    const float* bias;      // biases by distance (a table as in common.cuh, in log2 units), or null
+    int bias_reach;
 };
 
 // Whether pages come by TMA where the head size allows (the default) or by cp.async
@@ -564,7 +584,7 @@ extern "C" void bc_attention_decode_set_tma(int on) { g_ad_tma = on != 0; }
 static int g_ad_cluster16 = 1;
 extern "C" void bc_attention_decode_set_cluster16(int on) { g_ad_cluster16 = on != 0; }
 
-template <int D, bool TMA>
+template <int D, bool TMA, bool BIAS>
 static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, int q_stride, const void* k_cache, const void* v_cache,
                      const int* page_table, const int* row_pos, const int* row_slot, void* out, float* scratch, int* counters, int rows, int H,
                      int G, int max_pages, int n_pages, int window, float scale, int n_splits, FusedRope fr, cudaStream_t s) {
@@ -573,7 +593,7 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
     constexpr int SMEM = (AD_STAGES * 2 * TILE_BYTES > MERGE_BYTES ? AD_STAGES * 2 * TILE_BYTES : MERGE_BYTES) + 1024;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, TMA>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, TMA, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
         if (e != cudaSuccess) {
             bc_set_error("attention_decode: cannot set shared memory to %d: %s", SMEM, cudaGetErrorString(e));
             return (int)e;
@@ -592,7 +612,7 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
         static int sixteen = -1;
         if (sixteen < 0) {
             sixteen = 0;
-            if (cudaFuncSetAttribute(attention_decode_kernel<D, TMA>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
+            if (cudaFuncSetAttribute(attention_decode_kernel<D, TMA, BIAS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
                 cudaLaunchConfig_t cfg = {};
                 cfg.gridDim = dim3(16, 1, 1);
                 cfg.blockDim = dim3(TMA ? AD_THREADS_TMA : AD_THREADS);
@@ -604,7 +624,7 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
                 cfg.attrs = attr;
                 cfg.numAttrs = 1;
                 int fit = 0;
-                if (cudaOccupancyMaxActiveClusters(&fit, attention_decode_kernel<D, TMA>, &cfg) == cudaSuccess && fit > 0) sixteen = 1;
+                if (cudaOccupancyMaxActiveClusters(&fit, attention_decode_kernel<D, TMA, BIAS>, &cfg) == cudaSuccess && fit > 0) sixteen = 1;
             }
             (void)cudaGetLastError();
         }
@@ -613,15 +633,15 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
     if (n_splits > 8 && csize < n_splits && !(scratch && counters)) csize = 1;
     const bool clustered = n_splits > 1 && fr.allow_cluster && csize > 1;
     if (clustered)
-        bc_launch_clustered(attention_decode_kernel<D, TMA>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, dim3(csize, 1, 1), mk, mv, (const bf16*)q,
+        bc_launch_clustered(attention_decode_kernel<D, TMA, BIAS>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, dim3(csize, 1, 1), mk, mv, (const bf16*)q,
                             q_stride, (const bf16*)k_cache, (const bf16*)v_cache, page_table, row_pos, row_slot, (bf16*)out, scratch, counters, H, G,
                             max_pages, n_pages, window, scale * 1.4426950408889634f, (const float2*)fr.cos_sin, fr.pairing, fr.fuse,
-                            fr.k_off, fr.v_off, (bf16*)k_cache, (bf16*)v_cache, csize, fr.sink, fr.out_scale);
+                            fr.k_off, fr.v_off, (bf16*)k_cache, (bf16*)v_cache, csize, fr.sink, fr.out_scale, fr.bias, fr.bias_reach);
     else
-        bc_launch(attention_decode_kernel<D, TMA>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, mk, mv, (const bf16*)q, q_stride, (const bf16*)k_cache,
+        bc_launch(attention_decode_kernel<D, TMA, BIAS>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, mk, mv, (const bf16*)q, q_stride, (const bf16*)k_cache,
                   (const bf16*)v_cache, page_table, row_pos, row_slot, (bf16*)out, scratch, counters, H, G, max_pages, n_pages, window,
                   scale * 1.4426950408889634f, (const float2*)fr.cos_sin, fr.pairing, fr.fuse, fr.k_off, fr.v_off, (bf16*)k_cache,
-                  (bf16*)v_cache, 0, fr.sink, fr.out_scale);
+                  (bf16*)v_cache, 0, fr.sink, fr.out_scale, fr.bias, fr.bias_reach);
     BC_LAUNCH_STATUS();
 }
 
@@ -637,12 +657,16 @@ static int launch(const void* q, int q_stride, const void* k_cache, const void* 
             int st = bc_cached_cache_map(&mk, k_cache, cache_rows, D, "attention_decode");
             if (st == BC_OK) st = bc_cached_cache_map(&mv, v_cache, cache_rows, D, "attention_decode");
             if (st != BC_OK) return st;
-            return launch_as<D, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
-                                      max_pages, n_pages, window, scale, n_splits, fr, s);
+            return fr.bias ? launch_as<D, true, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H,
+                                                      G, max_pages, n_pages, window, scale, n_splits, fr, s)
+                           : launch_as<D, true, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H,
+                                                       G, max_pages, n_pages, window, scale, n_splits, fr, s);
         }
     }
-    return launch_as<D, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, max_pages,
-                               n_pages, window, scale, n_splits, fr, s);
+    return fr.bias ? launch_as<D, false, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
+                                               max_pages, n_pages, window, scale, n_splits, fr, s)
+                   : launch_as<D, false, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
+                                                max_pages, n_pages, window, scale, n_splits, fr, s);
 }
 
 // Whether this kernel takes the sizes (else the caller uses the one-warp-a-row kernel).
@@ -667,7 +691,8 @@ extern "C" int bc_attention_decode_workspace(int rows, int H, int G, int D, int 
 static int decode_fused(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table, const int* row_pos,
                         const int* row_slot, void* out, float* scratch, int* counters, int rows, int H, int G, int D, int max_pages, int n_pages,
                         int window, float scale, int n_splits, const float* cos_sin, int pairing, int fuse, int sink, float out_scale,
-                        cudaStream_t s) {
+                        const float* bias, int bias_reach, cudaStream_t s) {
+    BC_CHECK_ARG(bias == nullptr || bias_reach > 0, "attention_decode: a table of biases for %d distances", bias_reach);
     BC_CHECK_ARG(rows >= 0 && rows <= 65535, "attention_decode: %d rows (at most 65535)", rows);
     BC_CHECK_ARG(bc_attention_decode_accepts(H, G, D), "attention_decode: H=%d G=%d D=%d is outside what this kernel takes "
                  "(at most %d heads a kv head, head size a multiple of 16 up to 128)", H, G, D, AD_MAX_GROUP);
@@ -678,7 +703,7 @@ static int decode_fused(const void* q, int q_stride, const void* k_cache, const 
     BC_CHECK_ARG((fuse & 3) == 0 || q_stride == (H + 2 * G) * D, "attention_decode: fused mode wants the fused projection, stride %d", (H + 2 * G) * D);
     BC_CHECK_ARG((fuse & 3) == 0 || cos_sin == nullptr || (uintptr_t)cos_sin % 16 == 0, "attention_decode: the rotary table must be 16-byte aligned");
     if (rows == 0) return BC_OK;
-    FusedRope fr{cos_sin, pairing, fuse & 3, H * D, (H + G) * D, (fuse & 4) == 0, sink, out_scale};
+    FusedRope fr{cos_sin, pairing, fuse & 3, H * D, (H + G) * D, (fuse & 4) == 0, sink, out_scale, bias, bias_reach};
 #define AD_CASE(DD) \
     case DD: return launch<DD>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, max_pages, n_pages, window, scale, n_splits, fr, s);
     switch (D) {
@@ -694,18 +719,19 @@ extern "C" int bc_attention_decode_fused_bf16(const void* q, int q_stride, const
                                               int H, int G, int D, int max_pages, int n_pages, int window, float scale, int n_splits,
                                               const float* cos_sin, int pairing, int fuse, cudaStream_t s) {
     return decode_fused(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, D, max_pages, n_pages, window,
-                        scale, n_splits, cos_sin, pairing, fuse, 0, 1.0f, s);
+                        scale, n_splits, cos_sin, pairing, fuse, 0, 1.0f, nullptr, 0, s);
 }
 
 // The plain kernel (q rotated already, the cache holding the row) with a sink (one more position of score 0 without a value,
-// counted once where a row's last sums are made) and a factor on the output; fuse: 0, or 4 to send the splits through scratch.
+// counted once where a row's last sums are made), a factor on the output and biases by distance (a table as in common.cuh, in log2
+// units, or null); fuse: 0, or 4 to send the splits through scratch.
 extern "C" int bc_attention_decode_sink_bf16(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                              const int* row_pos, const int* row_slot, void* out, float* scratch, int* counters, int rows,
                                              int H, int G, int D, int max_pages, int n_pages, int window, float scale, int n_splits, int fuse,
-                                             int sink, float out_scale, cudaStream_t s) {
+                                             int sink, float out_scale, const float* bias, int bias_reach, cudaStream_t s) {
     BC_CHECK_ARG((fuse & 3) == 0, "attention_decode: the sink comes with the plain kernel (fuse %d)", fuse);
     return decode_fused(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, D, max_pages, n_pages, window,
-                        scale, n_splits, nullptr, 0, fuse, sink, out_scale, s);
+                        scale, n_splits, nullptr, 0, fuse, sink, out_scale, bias, bias_reach, s);
 }
 
 // q: row r's head h at q + r * q_stride + h * D.  scratch / counters: see above; counters
@@ -750,7 +776,7 @@ static int launch_static(float* scratch, int* counters, const void* q, int q_str
         // First call for this head size on this device: let the kernel use the shared memory it needs.
         std::lock_guard<std::mutex> lock(g_static_mutex);
         if (!(g_static_configured[device] & (1u << (D / 16)))) {
-            cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+            cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
             if (e != cudaSuccess) {
                 bc_set_error("attention_decode_static: cannot set shared memory to %d: %s", SMEM, cudaGetErrorString(e));
                 return (int)e;
@@ -758,9 +784,9 @@ static int launch_static(float* scratch, int* counters, const void* q, int q_str
             g_static_configured[device] |= 1u << (D / 16);
         }
     }
-    bc_launch(attention_decode_kernel<D, false>, dim3(n_splits, G, rows), dim3(AD_THREADS), (size_t)SMEM, s, none, none, (const bf16*)q, q_stride,
+    bc_launch(attention_decode_kernel<D, false, false>, dim3(n_splits, G, rows), dim3(AD_THREADS), (size_t)SMEM, s, none, none, (const bf16*)q, q_stride,
               (const bf16*)k_cache, (const bf16*)v_cache, page_table, row_pos, row_slot, (bf16*)out, scratch, counters, H, G, max_pages,
-              n_pages, window, scale * 1.4426950408889634f, (const float2*)nullptr, 0, 0, 0, 0, (bf16*)nullptr, (bf16*)nullptr, 0, 0, 1.0f);
+              n_pages, window, scale * 1.4426950408889634f, (const float2*)nullptr, 0, 0, 0, 0, (bf16*)nullptr, (bf16*)nullptr, 0, 0, 1.0f, (const float*)nullptr, 0);
     BC_LAUNCH_STATUS();
 }
 

@@ -21,6 +21,9 @@
 //     operand is read out of tensor memory, into a TMEM accumulator that stays there for the
 //     whole block.  Values are the n-major B operand ([position][d] with d contiguous),
 //     exactly as TMA wrote the page.  Shared memory holds Q and the ring of pages, nothing else.
+//   - A table of biases by distance (common.cuh; BIAS) is added to the scores on their way to the exponentials: by the element in
+//     pages near a warp's rows (the lanes of a warp are consecutive rows, so their entries lie side by side), as one number a
+//     row where every distance of the page is past the table's reach.
 //   - The running maximum is only raised when the new maximum exceeds it by more than 8 (in
 //     log2 units), so P stays below 2^8 and the accumulator is rescaled (TMEM load, multiply,
 //     store) a few times a block instead of once a page.  Sums and outputs use the same
@@ -74,12 +77,13 @@ extern "C" int bc_attention_prefill_tc_set_trace(long long* buf, int y) {
 // two groups of softmax warps give every SM sub-partition two warps to switch between while
 // one waits for TMEM, a fence or a barrier: with one tile the softmax warps, one a
 // sub-partition, are the kernel's limit.  One tile serves steps with few new rows.
-template <int D, int DV, int NT>
+template <int D, int DV, int NT, bool BIAS>
 __global__ void __launch_bounds__(64 + NT * 128, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* __restrict__ page_table, const int* __restrict__ seq_rows,
                             const int* __restrict__ seq_slot, const int* __restrict__ seq_start, bf16* __restrict__ out, int H, int G,
-                            int max_pages, int n_pages, int window, int chunk, float scale_log2, int sink, const float* sink_values, float out_scale) {
+                            int max_pages, int n_pages, int window, int chunk, float scale_log2, int sink, const float* sink_values, float out_scale,
+                            const float* __restrict__ bias, int bias_reach) {
     constexpr int THREADS = 64 + NT * 128;
     constexpr int STAGES = APT_STAGES(D, NT);
     // P in shared memory only (APT_P_TMEM 0): two P tiles a query tile let the softmax of page
@@ -272,6 +276,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int warp_chunk_lo = chunk > 0 ? (start + tok0 + (t * APT_ROWS + 32 * q + 31) / group) / chunk * chunk : 0;
         const uint32_t lane_base = tmem + ((uint32_t)(32 * q) << 16);
         const uint32_t o_addr = lane_base + O_COL + t * D;
+        const float* my_bias = BIAS ? bias_of_kv_head(bias, bias_reach, group, g) + row % group : nullptr;     // this row's head at distance 0
+        const float far_bias = BIAS ? __ldg(my_bias + (size_t)(bias_reach - 1) * group) : 0.0f;
         float m_used = -INFINITY, l = 0.0f;
         bool ok = true;
         for (int j = 0; j < n_tiles; j++) {
@@ -291,6 +297,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // by all of its rows (padding rows are never written): no mask to work out.
             const bool whole = window == 0 && page_ok && tile * BC_PAGE + BC_PAGE - 1 <= warp_first_pos && tile * BC_PAGE >= warp_chunk_lo;
             float tmax = -INFINITY;
+            // Pages some of whose distances lie within the table's reach take their biases one by one, scaled scores and all; the others
+            // leave both to the exponentials' own multiply-add.
+            const bool near = BIAS && warp_first_pos - (tile * BC_PAGE + BC_PAGE - 1) < bias_reach - 1;
+            if (BIAS && near) {
+                const float* bp = my_bias + (ptrdiff_t)max(pos - tile * BC_PAGE, 0) * group;      // position 0 of the page; then one distance nearer each
+#pragma unroll
+                for (int c = 0; c < 64; c++) {
+                    sv[c] = __float_as_uint(fmaf(__uint_as_float(sv[c]), scale_log2, __ldg(bp)));
+                    bp -= group;
+                }
+            }
+            const float page_scale = BIAS && near ? 1.0f : scale_log2, page_bias = BIAS && !near ? far_bias : 0.0f;
             if (whole) {
                 // Two chains of three-input maxima: 32 instructions, each chain 16 long.
                 float ta = -INFINITY, tb = -INFINITY;
@@ -310,7 +328,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     tmax = fmaxf(tmax, v);
                 }
             }
-            const float m_true = fmaxf(m_used, tmax * scale_log2);
+            const float m_true = fmaxf(m_used, BIAS ? fmaf(tmax, page_scale, page_bias) : tmax * scale_log2);
             const bool raise = m_true > m_used + APT_RAISE;     // also the first finite maximum: -inf + 8 = -inf
             float corr = 1.0f;
             if (raise) {
@@ -352,7 +370,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const float base = m_used == -INFINITY ? 0.0f : m_used;
             // Scores scaled and shifted two at a time (fma.rn.f32x2: the same roundings as fmaf),
             // the exponentials' sums kept in four pairs, so that no chain of additions is longer than 8.
-            const uint64_t scale2 = pack_f32x2(scale_log2, scale_log2), shift2 = pack_f32x2(-base, -base);
+            const float shift = BIAS ? page_bias - base : -base;
+            const uint64_t scale2 = pack_f32x2(page_scale, page_scale), shift2 = pack_f32x2(shift, shift);
             uint64_t sums[4] = {0ull, 0ull, 0ull, 0ull};
 #if APT_P_TMEM
             // P goes back into tensor memory, two bf16 a column, over the scores just read (this
@@ -470,17 +489,17 @@ static int query_map(CUtensorMap* map, const void* q, int q_stride, int total_ro
     return BC_OK;
 }
 
-template <int D, int DV, int NT>
+template <int D, int DV, int NT, bool BIAS>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const int* page_table, const int* seq_rows,
                   const int* seq_slot, const int* seq_start, void* out, int seqs, int max_new, int H, int G, int max_pages, int n_pages,
-                  int window, int chunk, float scale, int sink, const float* sink_values, float out_scale, cudaStream_t s) {
+                  int window, int chunk, float scale, int sink, const float* sink_values, float out_scale, const float* bias, int bias_reach, cudaStream_t s) {
     constexpr int DB = D / 64;
     constexpr int STAGES = APT_STAGES(D, NT), PB = APT_PB(D, NT);
     constexpr int SMEM = DB * NT * APT_ROWS * 128 + NT * PB * APT_ROWS * 128 + STAGES * 2 * DB * BC_PAGE * 128 + 1024;
     static_assert(SMEM <= APT_SMEM_LIMIT, "the ring does not fit");
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D, DV, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D, DV, NT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
         if (e != cudaSuccess) {
             bc_set_error("attention_prefill_tc: cannot set shared memory to %d: %s", SMEM, cudaGetErrorString(e));
             return (int)e;
@@ -489,8 +508,9 @@ static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMa
     }
     const int tokens_per_block = NT * APT_ROWS / (H / G);
     dim3 grid(G, (max_new + tokens_per_block - 1) / tokens_per_block, seqs);
-    cudaError_t e = bc_launch(attention_prefill_tc_kernel<D, DV, NT>, grid, dim3(64 + NT * 128), (size_t)SMEM, s, mq, mk, mv, page_table, seq_rows,
-                              seq_slot, seq_start, (bf16*)out, H, G, max_pages, n_pages, window, chunk, scale * 1.4426950408889634f, sink, sink_values, out_scale);
+    cudaError_t e = bc_launch(attention_prefill_tc_kernel<D, DV, NT, BIAS>, grid, dim3(64 + NT * 128), (size_t)SMEM, s, mq, mk, mv, page_table, seq_rows,
+                              seq_slot, seq_start, (bf16*)out, H, G, max_pages, n_pages, window, chunk, scale * 1.4426950408889634f, sink, sink_values, out_scale,
+                              bias, bias_reach);
     if (e != cudaSuccess) {
         bc_set_error("attention_prefill_tc: launch failed: %s", cudaGetErrorString(e));
         return (int)e;
@@ -527,7 +547,9 @@ extern "C" int bc_attention_prefill_tc_accepts_kv(int H, int G, int D, int DV) {
 // q and the caches 16-byte aligned, q_stride a multiple of 8.
 static int prefill_tc(const void* q, int q_stride, int total_rows, const void* k_cache, const void* v_cache, const int* page_table,
                       const int* seq_rows, const int* seq_slot, const int* seq_start, void* out, int seqs, int max_new, int H, int G, int D, int DV,
-                      int max_pages, int n_pages, int window, int chunk, float scale, int sink, const float* sink_values, float out_scale, cudaStream_t s) {
+                      int max_pages, int n_pages, int window, int chunk, float scale, int sink, const float* sink_values, float out_scale, const float* bias, int bias_reach,
+                      cudaStream_t s) {
+    BC_CHECK_ARG(bias == nullptr || bias_reach > 0, "attention_prefill_tc: a table of biases for %d distances", bias_reach);
     BC_CHECK_ARG(seqs >= 0 && seqs <= 65535 && max_new >= 0 && total_rows >= 0, "attention_prefill_tc: bad sizes seqs=%d max_new=%d rows=%d", seqs,
                  max_new, total_rows);
     BC_CHECK_ARG(bc_attention_prefill_tc_accepts_kv(H, G, D, DV), "attention_prefill_tc: H=%d G=%d D=%d DV=%d is outside what this kernel takes "
@@ -549,7 +571,8 @@ static int prefill_tc(const void* q, int q_stride, int total_rows, const void* k
     const long long cache_rows = (long long)n_pages * G * BC_PAGE;
     if ((st = bc_cached_cache_map(&mk, k_cache, cache_rows, D, "attention_prefill_tc")) != BC_OK) return st;
     if ((st = bc_cached_cache_map(&mv, v_cache, cache_rows, DV, "attention_prefill_tc")) != BC_OK) return st;
-#define APT_GO(DD, VV, NN) return launch<DD, VV, NN>(mq, mk, mv, page_table, seq_rows, seq_slot, seq_start, out, seqs, max_new, H, G, max_pages, n_pages, window, chunk, scale, sink, sink_values, out_scale, s)
+#define APT_AS(DD, VV, NN, BB) return launch<DD, VV, NN, BB>(mq, mk, mv, page_table, seq_rows, seq_slot, seq_start, out, seqs, max_new, H, G, max_pages, n_pages, window, chunk, scale, sink, sink_values, out_scale, bias, bias_reach, s)
+#define APT_GO(DD, VV, NN) do { if (bias) APT_AS(DD, VV, NN, true); APT_AS(DD, VV, NN, false); } while (0)
     if (D == 64 && nt == 1) APT_GO(64, 64, 1);
     if (D == 64) APT_GO(64, 64, 2);
     if (DV == 64 && nt == 1) APT_GO(128, 64, 1);
@@ -557,6 +580,7 @@ static int prefill_tc(const void* q, int q_stride, int total_rows, const void* k
     if (nt == 1) APT_GO(128, 128, 1);
     APT_GO(128, 128, 2);
 #undef APT_GO
+#undef APT_AS
 }
 
 extern "C" int bc_attention_prefill_tc_bf16(const void* q, int q_stride, int total_rows, const void* k_cache, const void* v_cache,
@@ -564,16 +588,18 @@ extern "C" int bc_attention_prefill_tc_bf16(const void* q, int q_stride, int tot
                                             int seqs, int max_new, int H, int G, int D, int DV, int max_pages, int n_pages, int window,
                                             int chunk, float scale, cudaStream_t s) {
     return prefill_tc(q, q_stride, total_rows, k_cache, v_cache, page_table, seq_rows, seq_slot, seq_start, out, seqs, max_new, H, G, D, DV, max_pages,
-                      n_pages, window, chunk, scale, 0, nullptr, 1.0f, s);
+                      n_pages, window, chunk, scale, 0, nullptr, 1.0f, nullptr, 0, s);
 }
 
-// The same with a sink (one more position without a value, of score 0 or of sink_values[head] if that is not null) and a factor on the output.
+// The same with a sink (one more position without a value, of score 0 or of sink_values[head] if that is not null), a factor on the output and
+// biases by distance: a table as in common.cuh, in log2 units (null: none).
 extern "C" int bc_attention_prefill_tc_sink_bf16(const void* q, int q_stride, int total_rows, const void* k_cache, const void* v_cache,
                                                  const int* page_table, const int* seq_rows, const int* seq_slot, const int* seq_start, void* out,
                                                  int seqs, int max_new, int H, int G, int D, int DV, int max_pages, int n_pages, int window,
-                                                 int chunk, float scale, int sink, const float* sink_values, float out_scale, cudaStream_t s) {
+                                                 int chunk, float scale, int sink, const float* sink_values, float out_scale, const float* bias, int bias_reach,
+                                                 cudaStream_t s) {
     return prefill_tc(q, q_stride, total_rows, k_cache, v_cache, page_table, seq_rows, seq_slot, seq_start, out, seqs, max_new, H, G, D, DV, max_pages,
-                      n_pages, window, chunk, scale, sink, sink_values, out_scale, s);
+                      n_pages, window, chunk, scale, sink, sink_values, out_scale, bias, bias_reach, s);
 }
 
 // This unit's status word (0, or where a bounded wait gave up), its wait limit and its word

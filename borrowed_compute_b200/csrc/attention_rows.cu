@@ -5,6 +5,7 @@
 // sliding window), or the first position of p's chunk, floor(p / chunk) * chunk (chunks are
 // counted from the sequence's position 0), whichever is later:
 //   s_t = (q . k_t) * scale;  out = sum_t softmax(s)_t v_t
+// Where a table of biases by distance is given (see common.cuh), the head's number for p - t is added to s_t.
 // Keys have D values a head and values DV, which may differ.
 // (crates/bc-infer/src/model.rs:448-481).  Like the reference's kernel
 // (crates/bc-infer/src/gpu/kernels.h:271-324) it keeps a running maximum m, a running sum
@@ -63,7 +64,8 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_kernel(const T* __r
                                                                    const T* __restrict__ v_cache, const int* __restrict__ page_table,
                                                                    const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                                                                    T* __restrict__ out, int H, int G, int D, int DV, int max_pages,
-                                                                   int n_pages, int window, int chunk, float scale, int sink, float out_scale) {
+                                                                   int n_pages, int window, int chunk, float scale, int sink, float out_scale,
+                                                                   const float* __restrict__ bias, int bias_reach) {
     __shared__ __align__(16) float qs[WARPS][MAX_D];
     pdl_launch_dependents();
     pdl_wait();
@@ -81,6 +83,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_kernel(const T* __r
     }
     const int pos = row_pos[r];
     const int g = h / (H / G);
+    const float* hb = bias == nullptr ? nullptr : bias_of_kv_head(bias, bias_reach, H / G, g) + h % (H / G);
     const T* qh = q + (size_t)r * q_stride + (size_t)h * D;
     for (int d = lane; d < D; d += 32) qs[warp][d] = to_f32(qh[d]);
     __syncwarp();
@@ -103,6 +106,7 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_kernel(const T* __r
         const bool seen = page >= 0 && t >= lo && t <= pos;
         float s = -INFINITY;
         if (seen) s = (D % 8 == 0 ? KeyDot<T>::dot(k_cache + base + (size_t)lane * D, qs[warp], D) : dot_any<T>(k_cache + base + (size_t)lane * D, qs[warp], D)) * scale;
+        if (seen && hb != nullptr) s += hb[(size_t)min(pos - t, bias_reach - 1) * (H / G)];
         const float mn = fmaxf(m, warp_max(s));
         const float corr = mn == -INFINITY ? 1.0f : expf(m - mn);
         const float p = seen ? expf(s - mn) : 0.0f;
@@ -134,7 +138,8 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_kernel(const T* __r
 template <class T>
 static int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table, const int* row_pos,
                   const int* row_slot, void* out, int rows, int H, int G, int D, int DV, int max_pages, int n_pages, int window, int chunk,
-                  float scale, int sink, float out_scale, cudaStream_t s) {
+                  float scale, int sink, float out_scale, const float* bias, int bias_reach, cudaStream_t s) {
+    BC_CHECK_ARG(bias == nullptr || bias_reach > 0, "attention_rows: a table of biases for %d distances", bias_reach);
     BC_CHECK_ARG(rows >= 0 && H > 0 && G > 0 && H % G == 0, "attention_rows: bad sizes rows=%d H=%d G=%d", rows, H, G);
     BC_CHECK_ARG(D > 0 && D <= MAX_D, "attention_rows: head size %d is not within 1 to %d", D, MAX_D);
     BC_CHECK_ARG(DV > 0 && DV <= MAX_D && window >= 0 && chunk >= 0, "attention_rows: bad value width %d, window %d or chunk %d", DV, window, chunk);
@@ -142,7 +147,7 @@ static int launch(const void* q, int q_stride, const void* k_cache, const void* 
     if (rows == 0) return BC_OK;
     dim3 grid(rows, (H + WARPS - 1) / WARPS);
     bc_launch(attention_rows_kernel<T>, grid, dim3(WARPS * 32), 0, s, (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, page_table,
-              row_pos, row_slot, (T*)out, H, G, D, DV, max_pages, n_pages, window, chunk, scale, sink, out_scale);
+              row_pos, row_slot, (T*)out, H, G, D, DV, max_pages, n_pages, window, chunk, scale, sink, out_scale, bias, bias_reach);
     BC_LAUNCH_STATUS();
 }
 
@@ -150,35 +155,38 @@ static int launch(const void* q, int q_stride, const void* k_cache, const void* 
 extern "C" int bc_attention_rows_f32(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                      const int* row_pos, const int* row_slot, void* out, int rows, int H, int G, int D, int max_pages,
                                      int n_pages, int window, float scale, cudaStream_t s) {
-    return launch<float>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, D, max_pages, n_pages, window, 0, scale, 0, 1.0f, s);
+    return launch<float>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, D, max_pages, n_pages, window, 0, scale, 0, 1.0f, nullptr, 0, s);
 }
 extern "C" int bc_attention_rows_bf16(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                       const int* row_pos, const int* row_slot, void* out, int rows, int H, int G, int D, int max_pages,
                                       int n_pages, int window, float scale, cudaStream_t s) {
-    return launch<bf16>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, D, max_pages, n_pages, window, 0, scale, 0, 1.0f, s);
+    return launch<bf16>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, D, max_pages, n_pages, window, 0, scale, 0, 1.0f, nullptr, 0, s);
 }
 
 // The same with values of their own width DV (out: [rows, H, DV]) and a chunk mask beside the window (0: none).
 extern "C" int bc_attention_rows_kv_f32(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                         const int* row_pos, const int* row_slot, void* out, int rows, int H, int G, int D, int DV, int max_pages,
                                         int n_pages, int window, int chunk, float scale, cudaStream_t s) {
-    return launch<float>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, 0, 1.0f, s);
+    return launch<float>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, 0, 1.0f, nullptr, 0, s);
 }
 extern "C" int bc_attention_rows_kv_bf16(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                          const int* row_pos, const int* row_slot, void* out, int rows, int H, int G, int D, int DV, int max_pages,
                                          int n_pages, int window, int chunk, float scale, cudaStream_t s) {
-    return launch<bf16>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, 0, 1.0f, s);
+    return launch<bf16>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, 0, 1.0f, nullptr, 0, s);
 }
 
 // The same with a sink (one more position of score 0 without a value, so that the weights of a row add up to less
-// than one) and a factor on the output.
+// than one), a factor on the output, and biases by distance: a table as in common.cuh
+// (null: none).
 extern "C" int bc_attention_rows_sink_f32(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                           const int* row_pos, const int* row_slot, void* out, int rows, int H, int G, int D, int DV, int max_pages,
-                                          int n_pages, int window, int chunk, float scale, int sink, float out_scale, cudaStream_t s) {
-    return launch<float>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, sink, out_scale, s);
+                                          int n_pages, int window, int chunk, float scale, int sink, float out_scale, const float* bias, int bias_reach,
+                                          cudaStream_t s) {
+    return launch<float>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, sink, out_scale, bias, bias_reach, s);
 }
 extern "C" int bc_attention_rows_sink_bf16(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                            const int* row_pos, const int* row_slot, void* out, int rows, int H, int G, int D, int DV, int max_pages,
-                                           int n_pages, int window, int chunk, float scale, int sink, float out_scale, cudaStream_t s) {
-    return launch<bf16>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, sink, out_scale, s);
+                                           int n_pages, int window, int chunk, float scale, int sink, float out_scale, const float* bias, int bias_reach,
+                                          cudaStream_t s) {
+    return launch<bf16>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, rows, H, G, D, DV, max_pages, n_pages, window, chunk, scale, sink, out_scale, bias, bias_reach, s);
 }

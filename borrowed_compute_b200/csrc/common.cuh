@@ -39,6 +39,17 @@ extern "C" int bc_sm_count();   // streaming multiprocessors of the current devi
 
 typedef __nv_bfloat16 bf16;
 
+// A table of attention biases by distance: for each kv head and each distance the numbers of the heads that share it, side by side,
+//   [kv heads][BC_BIAS_FRONT + reach + BC_BIAS_BACK][heads a kv head] float,
+// the distance 0 at entry BC_BIAS_FRONT.  Every distance from reach - 1 on has the last entry's numbers.  The entries ahead of the
+// distance 0 (of positions that are masked) and behind the reach (copies of the last) let a kernel read a page's 64 positions
+// without a clamp.
+#define BC_BIAS_FRONT 64
+#define BC_BIAS_BACK 128
+__device__ __forceinline__ const float* bias_of_kv_head(const float* bias, int reach, int group, int g) {
+    return bias + ((size_t)g * (BC_BIAS_FRONT + reach + BC_BIAS_BACK) + BC_BIAS_FRONT) * group;
+}
+
 // Programmatic dependent launch: a kernel launched with the attribute may start while its
 // predecessor in the stream is still draining.  Everything before pdl_wait() (set-up, and
 // loads of weights, which no kernel writes) then overlaps the predecessor's tail; pdl_wait()

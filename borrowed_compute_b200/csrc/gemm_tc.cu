@@ -988,6 +988,7 @@ struct TcGroupParams {
     int N, K;               // outputs a matrix and row, depth
     int matrix_rows;        // weight rows a matrix: N, or 2 N for SwiGLU (gate rows, then up rows)
     int stages;
+    float glu_limit, glu_alpha;   // SwiGLU: as in TcParams
 };
 
 template <int BN, int EPI>
@@ -1102,7 +1103,7 @@ gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
                 if (n >= p.N) continue;
                 float r[16];
 #pragma unroll
-                for (int j = 0; j < 16; j++) r[j] = EPI == EPI_SWIGLU ? silu_mul(__uint_as_float(v[j]), __uint_as_float(u[j])) : epi_plain<EPI>(__uint_as_float(v[j]));
+                for (int j = 0; j < 16; j++) r[j] = EPI == EPI_SWIGLU ? glu_mul(__uint_as_float(v[j]), __uint_as_float(u[j]), p.glu_limit, p.glu_alpha) : epi_plain<EPI>(__uint_as_float(v[j]));
 #pragma unroll
                 for (int j = 0; j < 16; j++) {
                     if (cc + j >= t_count) break;
@@ -1153,10 +1154,10 @@ static int launch_grouped(const CUtensorMap& mw, const CUtensorMap& mx, TcGroupP
 }
 
 // X [rows, K] bf16, sorted by matrix; W [matrices, N, K] bf16 (gated: [matrices, 2 N, K], gate rows then up rows); out
-// [rows, N]: bf16 silu(gate) * up if gated (1), bf16 max(sum, 0)^2 if gated is 2, else float.  table: [0] tiles; then, a tile, matrix, first row, rows (at most
+// [rows, N]: bf16 silu(gate) * up if gated (1; with glu_limit > 0 the bounded gate of bc_gemm_tc_glu_bf16), bf16 max(sum, 0)^2 if gated is 2, else float.  table: [0] tiles; then, a tile, matrix, first row, rows (at most
 // tile_rows, one of 16, 32, 64, 128, 256); max_tiles: the most tiles the table can hold.  K a multiple of 8.
 extern "C" int bc_gemm_tc_grouped_bf16(const void* X, const void* W, void* out, const int* table, int rows, int matrices, int N, int K, int gated,
-                                       int tile_rows, int max_tiles, cudaStream_t s) {
+                                       int tile_rows, int max_tiles, float glu_limit, float glu_alpha, cudaStream_t s) {
     BC_CHECK_ARG(rows >= 0 && matrices > 0 && N > 0 && K > 0, "gemm_tc_grouped: bad sizes rows=%d matrices=%d N=%d K=%d", rows, matrices, N, K);
     BC_CHECK_ARG(K % 8 == 0, "gemm_tc_grouped: K=%d is not a multiple of 8 (TMA needs 16-byte row strides)", K);
     BC_CHECK_ARG(((uintptr_t)X % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc_grouped: operands must be 16-byte aligned");
@@ -1177,6 +1178,8 @@ extern "C" int bc_gemm_tc_grouped_bf16(const void* X, const void* W, void* out, 
     p.K = K;
     p.matrix_rows = matrix_rows;
     p.stages = 0;
+    p.glu_limit = glu_limit;
+    p.glu_alpha = glu_alpha;
 #define GROUPED(BN)                                                                         \
     case BN:                                                                                \
         return gated == 1 ? launch_grouped<BN, EPI_SWIGLU>(mw, mx, p, max_tiles, s)                \

@@ -2,13 +2,18 @@
 //
 //   route      z = W_router h in float; score s = sigmoid(z) (or softmax over the experts); the `top` largest scores of a
 //              row choose its experts (the lower index wins a tie); weights are the scores, as they are or divided by their sum
+//              Variations: a correction added to the scores for the choice alone; neighbouring experts in groups, of which only the best
+//              few can be chosen (a group is as good as its best choice score); identity experts, the router's last outputs, whose
+//              result is the input itself: they are chosen and weighed like the others and never sorted or multiplied
 //   count, offsets, fill
 //              rows sorted by expert: perm[j] = the (row, choice) pair at sorted place j, place[row * top + c] = its place,
 //              and a table of tiles of MOE_BM sorted rows that lie in one expert each
 //   gate_up    act[j] = silu(w g) * (w u) with g = W_gate^e x, u = W_up^e x, x the pair's row, w its weight: the weight
 //              multiplies the expert's input (weight_on_input), or act[j] = silu(g) * u and the weight waits for combine
 //   down       y[j] = W_down^e act[j] in float
-//   combine    residual[r] += sum over r's choices, in the order of choice, of y[place] (times the weight if it waited)
+//              (or, with a bound: act[j] = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit))
+//   combine    residual[r] += sum over r's choices, in the order of choice, of y[place] (times the weight if it waited); an identity
+//              expert's share is weight * h[r]
 //
 // Every sum of a row runs in an order that the sizes alone fix, and no two blocks add into one place: a row's result is the
 // same bits in any batch and at every repeat.  The products here run on the CUDA cores in float (the true 32-bit path, and
@@ -72,11 +77,13 @@ moe_logits_kernel(const T* __restrict__ h, const float* __restrict__ router, flo
     }
 }
 
-// One warp a row: the `top` largest logits (the lower index wins a tie) and their scores.
+// One warp a row: the `top` largest logits (the lower index wins a tie) and their scores.  CORRECTED: the largest scores plus
+// `correction` within the best `keep` of `groups` groups of neighbours (a group's rank is the largest of its members').
+template <bool CORRECTED>
 __global__ void __launch_bounds__(128)
 moe_choose_kernel(const float* __restrict__ logits, const int* __restrict__ row_slot, int* __restrict__ choice, float* __restrict__ weight, int rows,
-                  int E, int top, int softmax, int renorm, float factor) {
-    extern __shared__ float score_all[];                    // [4][E]
+                  int E, int top, int softmax, int renorm, float factor, const float* __restrict__ correction, int groups, int keep) {
+    extern __shared__ float score_all[];                    // [4][E], CORRECTED: then [4][groups]
     pdl_launch_dependents_if_resident();
     pdl_wait();
     PDL_FRESH(logits);
@@ -105,6 +112,44 @@ moe_choose_kernel(const float* __restrict__ logits, const int* __restrict__ row_
         for (int e = lane; e < E; e += 32) total += expf(score[e] - zmax);
         total = warp_sum(total);
     }
+    if (CORRECTED) {
+        // From here on the table holds what the choice goes by.
+        for (int e = lane; e < E; e += 32) {
+            const float s = softmax ? expf(score[e] - zmax) / total : 1.0f / (1.0f + expf(-score[e]));
+            score[e] = s + (correction != nullptr ? correction[e] : 0.0f);
+        }
+        __syncwarp();
+        if (keep < groups) {
+            float* best_of = score_all + 4 * E + warp * groups;
+            const int size = E / groups;
+            for (int g = lane; g < groups; g += 32) {
+                float b = -INFINITY;
+                for (int i = 0; i < size; i++) b = fmaxf(b, score[g * size + i]);
+                best_of[g] = b;
+            }
+            __syncwarp();
+            for (int k = 0; k < keep; k++) {
+                float best = -INFINITY;
+                int best_g = 0x7fffffff;
+                for (int g = lane; g < groups; g += 32) {
+                    const float z = best_of[g];
+                    if (z != INFINITY && (best_g == 0x7fffffff || z > best)) { best = z; best_g = g; }     // kept ones are marked +inf
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                    const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+                    if (og != 0x7fffffff && (best_g == 0x7fffffff || ob > best || (ob == best && og < best_g))) { best = ob; best_g = og; }
+                }
+                __syncwarp();
+                if (lane == 0 && best_g != 0x7fffffff) best_of[best_g] = INFINITY;
+                __syncwarp();
+            }
+            for (int e = lane; e < E; e += 32)
+                if (best_of[e / size] != INFINITY) score[e] = INFINITY;      // as if taken
+            __syncwarp();
+        }
+    }
     float picked_sum = 0.0f, mine = 0.0f;
     int mine_e = -1;
     for (int c = 0; c < top; c++) {
@@ -121,6 +166,10 @@ moe_choose_kernel(const float* __restrict__ logits, const int* __restrict__ row_
             if (oe != 0x7fffffff && (best_e == 0x7fffffff || ob > best || (ob == best && oe < best_e))) { best = ob; best_e = oe; }
         }
         if (best_e == 0x7fffffff) best_e = 0;
+        if (CORRECTED) {
+            best = logits[(size_t)r * E + best_e];
+            best = best == best ? best : -INFINITY;
+        }
         const float s = softmax ? expf(best - zmax) / total : 1.0f / (1.0f + expf(-best));
         picked_sum += s;
         if (lane == c) { mine = s; mine_e = best_e; }
@@ -282,7 +331,7 @@ template <class T, bool GATED>
 __global__ void __launch_bounds__(128)
 moe_product_kernel(const T* __restrict__ X, const T* __restrict__ W, const int* __restrict__ table, const int* __restrict__ perm,
                    const float* __restrict__ weight, T* __restrict__ out_act, float* __restrict__ out_f32, int N, int K, int top,
-                   int weight_on_input) {
+                   int weight_on_input, float limit, float alpha) {
     __shared__ float As[MOE_BK][MOE_BN + 4];       // only MOE_BM columns used
     __shared__ float Bs[MOE_BK][MOE_BN + 4];
     __shared__ float Cs[GATED ? MOE_BK : 1][MOE_BN + 4];
@@ -345,8 +394,13 @@ moe_product_kernel(const T* __restrict__ X, const T* __restrict__ W, const int* 
             if (n >= N) continue;
             const size_t o = (size_t)(j0 + r) * N + n;
             if (GATED) {
-                const float g = acc[i][j] * row_w[r], u = acc2[GATED ? i : 0][j] * row_w[r];
-                out_act[o] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+                float g = acc[i][j] * row_w[r], u = acc2[GATED ? i : 0][j] * row_w[r], a = 1.0f;
+                if (limit > 0.0f) {
+                    g = fminf(g, limit);
+                    u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+                    a = alpha;
+                }
+                out_act[o] = from_f32<T>(g / (1.0f + expf(-a * g)) * u);
             } else {
                 out_f32[o] = acc[i][j];
             }
@@ -377,28 +431,42 @@ moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ perm, const i
 }
 
 // ------------------------------------------------------------------------------------ combine
+// IDENTITY: choices from `experts` on are the row of h itself.  Their shares are one number a row times h[r]: their weights' sum.
+template <class T, bool IDENTITY>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ choice, const int* __restrict__ place, const float* __restrict__ weight,
-                   float* __restrict__ residual, int E, int top, int weight_on_output) {
+                   float* __restrict__ residual, int E, int top, int weight_on_output, const T* __restrict__ h, int experts) {
     __shared__ int where[MOE_MAX_TOP];
     __shared__ float factor[MOE_MAX_TOP];
     pdl_launch_dependents_if_resident();
     pdl_wait();
-    PDL_FRESH(y); PDL_FRESH(choice); PDL_FRESH(place); PDL_FRESH(weight);
+    PDL_FRESH(y); PDL_FRESH(choice); PDL_FRESH(place); PDL_FRESH(weight); PDL_FRESH(h);
     const int r = blockIdx.x;
+    __shared__ float own[MOE_MAX_TOP];       // weights of the identity experts among the choices, else 0
     // The row's places first, so that the loads of a column's values do not each wait for one.
     if ((int)threadIdx.x < top) {
-        const bool chosen = choice[(size_t)r * top + threadIdx.x] >= 0;
+        const int e = choice[(size_t)r * top + threadIdx.x];
+        const bool identity = IDENTITY && e >= experts;
+        const bool chosen = e >= 0 && !identity;
+        if (IDENTITY) own[threadIdx.x] = identity ? weight[(size_t)r * top + threadIdx.x] : 0.0f;
         where[threadIdx.x] = chosen ? place[(size_t)r * top + threadIdx.x] : -1;
         factor[threadIdx.x] = weight_on_output ? weight[(size_t)r * top + threadIdx.x] : 1.0f;
     }
     __syncthreads();
     bool any = false;
-    for (int i = 0; i < top; i++) any = any || where[i] >= 0;
+    float self = 0.0f;
+    for (int i = 0; i < top; i++) {
+        any = any || where[i] >= 0 || (IDENTITY && own[i] != 0.0f);
+        if (IDENTITY) self += own[i];
+    }
     if (!any) return;
     if (E % 4 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)residual % 16 == 0) {
         for (int c = 4 * threadIdx.x; c < E; c += 4 * blockDim.x) {
             float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (IDENTITY && self != 0.0f) {
+                const T* hr = h + (size_t)r * E + c;
+                sum = make_float4(self * to_f32(hr[0]), self * to_f32(hr[1]), self * to_f32(hr[2]), self * to_f32(hr[3]));
+            }
 #pragma unroll 4
             for (int i = 0; i < top; i++) {
                 if (where[i] < 0) continue;
@@ -414,7 +482,7 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ choice, 
         return;
     }
     for (int c = threadIdx.x; c < E; c += blockDim.x) {
-        float sum = 0.0f;
+        float sum = IDENTITY ? self * to_f32(h[(size_t)r * E + c]) : 0.0f;
 #pragma unroll 4
         for (int i = 0; i < top; i++) {
             if (where[i] < 0) continue;
@@ -428,25 +496,31 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ choice, 
 // ------------------------------------------------------------------------------------ launchers
 template <class T>
 static int route(const void* h, const float* router, const int* row_slot, float* logits, int* choice, float* weight, int rows, int E, int K, int top,
-                 int softmax, int renorm, float factor, cudaStream_t s) {
+                 int softmax, int renorm, float factor, const float* correction, int n_groups, int keep, cudaStream_t s) {
+    BC_CHECK_ARG(n_groups >= 1 && E % n_groups == 0 && keep >= 1 && keep <= n_groups && top <= E / n_groups * keep, "moe_route: %d of %d groups of %d experts for %d choices", keep, n_groups, E, top);
     BC_CHECK_ARG(rows >= 0 && E > 0 && K > 0 && top > 0 && top <= E && top <= MOE_MAX_TOP && E <= 2048, "moe_route: bad sizes rows=%d E=%d K=%d top=%d", rows, E, K, top);
     if (rows == 0) return BC_OK;
     const int groups = (E + ROUTE_EXPERTS - 1) / ROUTE_EXPERTS;
     BC_CHECK_ARG(groups <= 65535, "moe_route: too many experts (%d)", E);
     bc_launch(moe_logits_kernel<T>, dim3((rows + ROUTE_ROWS - 1) / ROUTE_ROWS, groups), dim3(32 * ROUTE_EXPERTS), 0, s, (const T*)h, router, logits, rows, E, K);
-    bc_launch(moe_choose_kernel, dim3((rows + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), s, (const float*)logits, row_slot, choice, weight, rows,
-              E, top, softmax, renorm, factor);
+    if (correction != nullptr || keep < n_groups)
+        bc_launch(moe_choose_kernel<true>, dim3((rows + 3) / 4), dim3(128), (size_t)4 * (E + n_groups) * sizeof(float), s, (const float*)logits, row_slot,
+                  choice, weight, rows, E, top, softmax, renorm, factor, correction, n_groups, keep);
+    else
+        bc_launch(moe_choose_kernel<false>, dim3((rows + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), s, (const float*)logits, row_slot, choice,
+                  weight, rows, E, top, softmax, renorm, factor, correction, 1, 1);
     BC_LAUNCH_STATUS();
 }
 // h: [rows, K] of the activation type; router: [E, K] float; row_slot: [rows] (negative: a padding row; may be null);
-// logits: [rows, E] float (scratch); choice: [rows, top] int; weight: [rows, top] float, every weight times `factor`.
+// logits: [rows, E] float (scratch); choice: [rows, top] int; weight: [rows, top] float, every weight times `factor`; correction: [E]
+// float or null; the experts as `groups` groups of neighbours, of which a row chooses from `keep` (1 and 1: no groups).
 extern "C" int bc_moe_route_f32(const void* h, const float* router, const int* row_slot, float* logits, int* choice, float* weight, int rows, int E,
-                                int K, int top, int softmax, int renorm, float factor, cudaStream_t s) {
-    return route<float>(h, router, row_slot, logits, choice, weight, rows, E, K, top, softmax, renorm, factor, s);
+                                int K, int top, int softmax, int renorm, float factor, const float* correction, int groups, int keep, cudaStream_t s) {
+    return route<float>(h, router, row_slot, logits, choice, weight, rows, E, K, top, softmax, renorm, factor, correction, groups, keep, s);
 }
 extern "C" int bc_moe_route_bf16(const void* h, const float* router, const int* row_slot, float* logits, int* choice, float* weight, int rows, int E,
-                                 int K, int top, int softmax, int renorm, float factor, cudaStream_t s) {
-    return route<bf16>(h, router, row_slot, logits, choice, weight, rows, E, K, top, softmax, renorm, factor, s);
+                                 int K, int top, int softmax, int renorm, float factor, const float* correction, int groups, int keep, cudaStream_t s) {
+    return route<bf16>(h, router, row_slot, logits, choice, weight, rows, E, K, top, softmax, renorm, factor, correction, groups, keep, s);
 }
 
 extern "C" int bc_moe_max_tiles(int pairs, int E, int tile_rows) { return (pairs + tile_rows - 1) / tile_rows + E; }
@@ -470,7 +544,7 @@ extern "C" int bc_moe_plan(const int* choice, int pairs, int E, int tile_rows, i
 
 template <class T>
 static int products(int gated, const void* X, const void* W, const int* table, const int* perm, const float* weight, void* out, int pairs, int E,
-                    int N, int K, int top, int weight_on_input, cudaStream_t s) {
+                    int N, int K, int top, int weight_on_input, float limit, float alpha, cudaStream_t s) {
     BC_CHECK_ARG(pairs >= 0 && E > 0 && N > 0 && K > 0 && top > 0, "moe_product: bad sizes pairs=%d E=%d N=%d K=%d", pairs, E, N, K);
     if (pairs == 0) return BC_OK;
     const int tiles = bc_moe_max_tiles(pairs, E, MOE_BM);
@@ -478,20 +552,21 @@ static int products(int gated, const void* X, const void* W, const int* table, c
     dim3 grid((N + MOE_BN - 1) / MOE_BN, tiles);
     if (gated)
         bc_launch(moe_product_kernel<T, true>, grid, dim3(128), 0, s, (const T*)X, (const T*)W, table, perm, weight, (T*)out, (float*)nullptr, N, K,
-                  top, weight_on_input);
+                  top, weight_on_input, limit, alpha);
     else
         bc_launch(moe_product_kernel<T, false>, grid, dim3(128), 0, s, (const T*)X, (const T*)W, table, perm, weight, (T*)nullptr, (float*)out, N, K,
-                  top, 0);
+                  top, 0, 0.0f, 0.0f);
     BC_LAUNCH_STATUS();
 }
 // gated: X [rows, K], W [E, 2 N, K], out [pairs, N] of the activation type; else X [pairs, K], W [E, N, K], out [pairs, N] float.
+// limit > 0: the gated product's activation with bounds.
 extern "C" int bc_moe_product_f32(int gated, const void* X, const void* W, const int* table, const int* perm, const float* weight, void* out,
-                                  int pairs, int E, int N, int K, int top, int weight_on_input, cudaStream_t s) {
-    return products<float>(gated, X, W, table, perm, weight, out, pairs, E, N, K, top, weight_on_input, s);
+                                  int pairs, int E, int N, int K, int top, int weight_on_input, float limit, float alpha, cudaStream_t s) {
+    return products<float>(gated, X, W, table, perm, weight, out, pairs, E, N, K, top, weight_on_input, limit, alpha, s);
 }
 extern "C" int bc_moe_product_bf16(int gated, const void* X, const void* W, const int* table, const int* perm, const float* weight, void* out,
-                                   int pairs, int E, int N, int K, int top, int weight_on_input, cudaStream_t s) {
-    return products<bf16>(gated, X, W, table, perm, weight, out, pairs, E, N, K, top, weight_on_input, s);
+                                   int pairs, int E, int N, int K, int top, int weight_on_input, float limit, float alpha, cudaStream_t s) {
+    return products<bf16>(gated, X, W, table, perm, weight, out, pairs, E, N, K, top, weight_on_input, limit, alpha, s);
 }
 
 template <class T>
@@ -517,6 +592,25 @@ extern "C" int bc_moe_combine(const float* y, const int* choice, const int* plac
                               int weight_on_output, cudaStream_t s) {
     BC_CHECK_ARG(rows >= 0 && width > 0 && top > 0, "moe_combine: bad sizes rows=%d width=%d top=%d", rows, width, top);
     if (rows == 0) return BC_OK;
-    bc_launch(moe_combine_kernel, dim3(rows), dim3(width >= 1024 ? 256 : 128), 0, s, y, choice, place, weight, residual, width, top, weight_on_output);
+    bc_launch(moe_combine_kernel<float, false>, dim3(rows), dim3(width >= 1024 ? 256 : 128), 0, s, y, choice, place, weight, residual, width, top,
+              weight_on_output, (const float*)nullptr, 0);
     BC_LAUNCH_STATUS();
+}
+// The same where choices from `experts` on are identity experts: their share is their weight times h[r] (h: [rows, width] of the
+// activation type); the weights are on the output.
+template <class T>
+static int combine_identity(const float* y, const int* choice, const int* place, const float* weight, float* residual, const void* h, int rows, int width,
+                            int top, int experts, cudaStream_t s) {
+    BC_CHECK_ARG(rows >= 0 && width > 0 && top > 0 && top <= MOE_MAX_TOP && experts > 0, "moe_combine_identity: bad sizes rows=%d width=%d top=%d experts=%d", rows, width, top, experts);
+    if (rows == 0) return BC_OK;
+    bc_launch(moe_combine_kernel<T, true>, dim3(rows), dim3(width >= 1024 ? 256 : 128), 0, s, y, choice, place, weight, residual, width, top, 1, (const T*)h, experts);
+    BC_LAUNCH_STATUS();
+}
+extern "C" int bc_moe_combine_identity_f32(const float* y, const int* choice, const int* place, const float* weight, float* residual, const void* h,
+                                           int rows, int width, int top, int experts, cudaStream_t s) {
+    return combine_identity<float>(y, choice, place, weight, residual, h, rows, width, top, experts, s);
+}
+extern "C" int bc_moe_combine_identity_bf16(const float* y, const int* choice, const int* place, const float* weight, float* residual, const void* h,
+                                            int rows, int width, int top, int experts, cudaStream_t s) {
+    return combine_identity<bf16>(y, choice, place, weight, residual, h, rows, width, top, experts, s);
 }

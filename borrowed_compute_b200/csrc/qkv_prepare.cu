@@ -196,7 +196,8 @@ __global__ void __launch_bounds__(256)
 qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                          const float* __restrict__ cos_sin, int n_positions, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                          const int* __restrict__ page_table, int max_pages, int n_pages, T* __restrict__ q_out, T* __restrict__ k_cache,
-                         T* __restrict__ v_cache, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache) {
+                         T* __restrict__ v_cache, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache,
+                         float temp_coef, int temp_every) {
     pdl_launch_dependents_if_resident();
     pdl_wait();
     PDL_FRESH(qkv);
@@ -213,6 +214,8 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
     if (slot >= 0 && pos >= 0 && pos / BC_PAGE < max_pages) page = page_table[(size_t)slot * max_pages + pos / BC_PAGE];
     if (page >= n_pages) page = -1;
     const bool cache = write_cache && page >= 0;
+    // Queries grow with their position: times 1 + coef ln(floor((p + 1) / every) + 1).
+    const float warmth = temp_every > 0 && pos >= 0 ? 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1)) : 1.0f;
     const int units = half + (D - rot);          // pairs that turn, then single dimensions that pass
     for (int head = warp; head < H + G; head += warps) {
         const bool is_q = head < H;
@@ -224,6 +227,7 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
             ss = warp_sum(ss);
         }
         const float scale = normed ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
+        const float more = is_q ? warmth : 1.0f;
         T* dst = is_q ? q_out + (size_t)r * nq + (size_t)head * D
                       : k_cache + (((size_t)(cache ? page : 0) * G + (head - H)) * BC_PAGE + pos % BC_PAGE) * D;
         if (!is_q && !cache) continue;
@@ -237,11 +241,11 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
                     va = ra;
                     vb = rb;
                 }
-                dst[a] = from_f32<T>(va);
-                dst[b] = from_f32<T>(vb);
+                dst[a] = from_f32<T>(va * more);
+                dst[b] = from_f32<T>(vb * more);
             } else {
                 const int d = rot + (u - half);
-                dst[d] = from_f32<T>(xh[d] * (normed ? scale * wt[d] : 1.0f));
+                dst[d] = from_f32<T>(xh[d] * (normed ? scale * wt[d] : 1.0f) * more);
             }
         }
     }
@@ -256,7 +260,8 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
 template <class T>
 static int launch_heads(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_sin, int n_positions, const int* row_pos,
                         const int* row_slot, const int* page_table, int max_pages, int n_pages, void* q_out, void* k_cache, void* v_cache, int rows,
-                        int H, int G, int VG, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache, cudaStream_t s) {
+                        int H, int G, int VG, int D, int DV, int rot, int pairing, float eps, int normed, int write_cache, float temp_coef, int temp_every, cudaStream_t s) {
+    BC_CHECK_ARG(temp_every >= 0, "qkv_prepare_heads: a query temperature that changes every %d positions", temp_every);
     BC_CHECK_ARG(rows >= 0 && H > 0 && G >= 0 && VG >= 0 && (G > 0) == (VG > 0) && D > 0 && DV > 0, "qkv_prepare_heads: bad sizes rows=%d H=%d G=%d D=%d DV=%d", rows, H, G, D, DV);
     BC_CHECK_ARG(rot >= 0 && rot % 2 == 0 && rot <= D, "qkv_prepare_heads: %d rotated dimensions of a head of %d", rot, D);
     BC_CHECK_ARG(!normed || (q_weight && (k_weight || G == 0)), "qkv_prepare_heads: the norm needs its weights");
@@ -264,23 +269,23 @@ static int launch_heads(const float* qkv, const float* q_weight, const float* k_
     const int heads = H + G;
     const int threads = heads >= 8 ? 256 : heads >= 4 ? 128 : 64;      // by the row's heads alone
     bc_launch(qkv_prepare_heads_kernel<T>, dim3(rows), dim3(threads), 0, s, qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot,
-              page_table, max_pages, n_pages, (T*)q_out, (T*)k_cache, (T*)v_cache, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache);
+              page_table, max_pages, n_pages, (T*)q_out, (T*)k_cache, (T*)v_cache, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, temp_coef, temp_every);
     BC_LAUNCH_STATUS();
 }
 
 // As bc_qkv_prepare_*, without biases; q_weight and k_weight hold D values each; cos_sin: [n_positions, rot / 2, 2];
-// qkv: [rows, H D + G D + VG DV]; v_cache: [pages, VG, PAGE, DV].
+// qkv: [rows, H D + G D + VG DV]; v_cache: [pages, VG, PAGE, DV].  temp_every > 0: queries times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
 extern "C" int bc_qkv_prepare_heads_f32(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_sin, int n_positions,
                                         const int* row_pos, const int* row_slot, const int* page_table, int max_pages, int n_pages, void* q_out,
                                         void* k_cache, void* v_cache, int rows, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps,
-                                        int normed, int write_cache, cudaStream_t s) {
+                                        int normed, int write_cache, float temp_coef, int temp_every, cudaStream_t s) {
     return launch_heads<float>(qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot, page_table, max_pages, n_pages, q_out, k_cache,
-                               v_cache, rows, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, s);
+                               v_cache, rows, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, temp_coef, temp_every, s);
 }
 extern "C" int bc_qkv_prepare_heads_bf16(const float* qkv, const float* q_weight, const float* k_weight, const float* cos_sin, int n_positions,
                                          const int* row_pos, const int* row_slot, const int* page_table, int max_pages, int n_pages, void* q_out,
                                          void* k_cache, void* v_cache, int rows, int H, int G, int VG, int D, int DV, int rot, int pairing, float eps,
-                                         int normed, int write_cache, cudaStream_t s) {
+                                         int normed, int write_cache, float temp_coef, int temp_every, cudaStream_t s) {
     return launch_heads<bf16>(qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot, page_table, max_pages, n_pages, q_out, k_cache,
-                              v_cache, rows, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, s);
+                              v_cache, rows, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, temp_coef, temp_every, s);
 }

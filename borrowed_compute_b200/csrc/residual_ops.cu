@@ -3,7 +3,9 @@
 //
 //   norm_add     x[r] += y[r] / sqrt(mean(y[r]^2) + eps) * w          (y float: the sublayer's result)
 //   norm_add_norm   the same, then h[r] = x[r] / sqrt(mean(x[r]^2) + eps2) * w2 in the activation type for the sublayer that
-//                follows, and y[r] = 0 for its result: one kernel between the two sublayers of a block
+//                follows, and y[r] = 0 for its result: one kernel between the two sublayers of a block.  Without w2 the next sublayer
+//                reads the stream itself: h[r] = x[r] rounded
+//   enter_plain  h[r] = x[r] rounded to the activation type, y[r] = 0  (ahead of the first such sublayer)
 //   relu2        out = max(z, 0)^2 in the activation type               (z float: an up product)
 //   glu_clipped  out = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit), from z = [g | u] float
 //   gated_add    x[r] += sigmoid(g . h[r]) * y[r]                       (one number a row: a gate on a shared expert)
@@ -53,7 +55,7 @@ extern "C" int bc_norm_add_f32(const float* y, const float* w, float* x, int row
 }
 
 // A thread keeps its columns through both norms: it adds into x the columns whose squares it then sums.
-template <class T>
+template <class T, bool PLAIN>
 __global__ void norm_add_norm_kernel(float* y, const float* __restrict__ wb, float* x, const float* __restrict__ w2, T* __restrict__ h, int E, float eps_b,
                                      float eps_2) {
     __shared__ float scratch[32];
@@ -78,8 +80,13 @@ __global__ void norm_add_norm_kernel(float* y, const float* __restrict__ wb, flo
             o.x += v.x * f * g.x; o.y += v.y * f * g.y; o.z += v.z * f * g.z; o.w += v.w * f * g.w;
             *reinterpret_cast<float4*>(xr + c) = o;
             *reinterpret_cast<float4*>(yr + c) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (PLAIN) {
+                hr[c] = from_f32<T>(o.x); hr[c + 1] = from_f32<T>(o.y); hr[c + 2] = from_f32<T>(o.z); hr[c + 3] = from_f32<T>(o.w);
+                continue;
+            }
             t += o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w;
         }
+        if (PLAIN) return;
         t = block_sum(t, scratch);
         const float f2 = 1.0f / sqrtf(t / (float)E + eps_2);
         for (int c = 4 * threadIdx.x; c < E; c += 4 * blockDim.x) {
@@ -97,18 +104,22 @@ __global__ void norm_add_norm_kernel(float* y, const float* __restrict__ wb, flo
         const float o = xr[c] + yr[c] * f * wb[c];
         xr[c] = o;
         yr[c] = 0.0f;
+        if (PLAIN) hr[c] = from_f32<T>(o);
         t += o * o;
     }
+    if (PLAIN) return;
     t = block_sum(t, scratch);
     const float f2 = 1.0f / sqrtf(t / (float)E + eps_2);
     for (int c = threadIdx.x; c < E; c += blockDim.x) hr[c] = from_f32<T>(xr[c] * f2 * w2[c]);
 }
 
-// y: [rows, E] float, left as zeros; wb, w2: [E] float; x: [rows, E] float, changed in place; h: [rows, E] of the activation type.
+// y: [rows, E] float, left as zeros; wb, w2: [E] float (w2 null: h is x rounded); x: [rows, E] float, changed in place; h: [rows, E] of the activation type.
 template <class T> static int norm_add_norm(float* y, const float* wb, float* x, const float* w2, void* h, int rows, int E, float eps_b, float eps_2, cudaStream_t s) {
     BC_CHECK_ARG(rows >= 0 && E > 0 && eps_b > 0.0f && eps_2 > 0.0f, "norm_add_norm: bad sizes rows=%d E=%d eps=%g, %g", rows, E, (double)eps_b, (double)eps_2);
     if (rows == 0) return BC_OK;
-    bc_launch(norm_add_norm_kernel<T>, dim3(rows), dim3(pick(E % 4 == 0 ? E / 4 : E)), 0, s, y, wb, x, w2, (T*)h, E, eps_b, eps_2);
+    const dim3 block(pick(E % 4 == 0 ? E / 4 : E));
+    if (w2) bc_launch(norm_add_norm_kernel<T, false>, dim3(rows), block, 0, s, y, wb, x, w2, (T*)h, E, eps_b, eps_2);
+    else bc_launch(norm_add_norm_kernel<T, true>, dim3(rows), block, 0, s, y, wb, x, w2, (T*)h, E, eps_b, eps_2);
     BC_LAUNCH_STATUS();
 }
 extern "C" int bc_norm_add_norm_f32(float* y, const float* wb, float* x, const float* w2, void* h, int rows, int E, float eps_b, float eps_2, cudaStream_t s) {
@@ -117,6 +128,34 @@ extern "C" int bc_norm_add_norm_f32(float* y, const float* wb, float* x, const f
 extern "C" int bc_norm_add_norm_bf16(float* y, const float* wb, float* x, const float* w2, void* h, int rows, int E, float eps_b, float eps_2, cudaStream_t s) {
     return norm_add_norm<bf16>(y, wb, x, w2, h, rows, E, eps_b, eps_2, s);
 }
+
+template <class T>
+__global__ void enter_plain_kernel(const float* x, T* __restrict__ h, float* __restrict__ y, size_t n4, size_t n) {
+    pdl_launch_dependents_if_resident();
+    pdl_wait();
+    PDL_FRESH(x);
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += (size_t)gridDim.x * blockDim.x) {
+        const float4 v = *reinterpret_cast<const float4*>(x + 4 * i);
+        h[4 * i] = from_f32<T>(v.x); h[4 * i + 1] = from_f32<T>(v.y); h[4 * i + 2] = from_f32<T>(v.z); h[4 * i + 3] = from_f32<T>(v.w);
+        *reinterpret_cast<float4*>(y + 4 * i) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+    if (blockIdx.x == 0)
+        for (size_t i = 4 * n4 + threadIdx.x; i < n; i += blockDim.x) {
+            h[i] = from_f32<T>(x[i]);
+            y[i] = 0.0f;
+        }
+}
+// x, y: [rows, E] float (16-byte aligned); h: the same of the activation type.
+template <class T> static int enter_plain(const float* x, void* h, float* y, int rows, int E, cudaStream_t s) {
+    BC_CHECK_ARG(rows >= 0 && E > 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0, "enter_plain: bad sizes rows=%d E=%d or alignment", rows, E);
+    if (rows == 0) return BC_OK;
+    const size_t n = (size_t)rows * E;
+    const size_t blocks = (n / 4 + 255) / 256;
+    bc_launch(enter_plain_kernel<T>, dim3((unsigned)(blocks < 1 ? 1 : blocks < 65535 ? blocks : 65535)), dim3(256), 0, s, x, (T*)h, y, n / 4, n);
+    BC_LAUNCH_STATUS();
+}
+extern "C" int bc_enter_plain_f32(const float* x, void* h, float* y, int rows, int E, cudaStream_t s) { return enter_plain<float>(x, h, y, rows, E, s); }
+extern "C" int bc_enter_plain_bf16(const float* x, void* h, float* y, int rows, int E, cudaStream_t s) { return enter_plain<bf16>(x, h, y, rows, E, s); }
 
 template <class T>
 __global__ void relu2_kernel(const float* z, T* __restrict__ out, size_t n) {

@@ -40,6 +40,12 @@ class DecoderModel:
         for i, run in enumerate(spec.schedule):
             if run.enter is not None and not 0 <= run.enter[0] < len(self.junctions):
                 raise ValueError(f"schedule entry {i} enters junction {run.enter[0]}, the model has {len(self.junctions)}")
+        # Positions that the embedding adds in its own kernel; where a norm stands between the two, or a junction reads the embedding
+        # again, they stay apart.
+        self.position_joined = self.position is not None and self.embedding_norm is None and not spec.junctions and self.embedding.join(self.position)
+        # Runs whose block may leave the stream in the activation type for the next one.
+        self.hand_over = [i + 1 < len(spec.schedule) and spec.schedule[i + 1].enter is None and self.blocks[run.layer].enters_plain
+                          and self.blocks[spec.schedule[i + 1].layer].enters_plain for i, run in enumerate(spec.schedule)]
         self.final_norm = _build(NORMS, spec.final_norm)
         self.head = _build(HEADS, spec.head)
         self.rt: Optional[Runtime] = None
@@ -83,6 +89,9 @@ class DecoderModel:
             needs.append(None if mixer is None else mixer.cache_need())
             states.append(None if mixer is None else mixer.state_need())
             memory_of.append(run.memory_of)
+        need = self.embedding.cache_need()
+        if need is not None:        # one more entry, behind the runs'
+            needs, states, memory_of = needs + [need], states + [None], memory_of + [None]
         # A run that reads another's memory may see further back than its owner: the owner keeps what both read.
         for i, j in enumerate(memory_of):
             if j is not None and needs[j] is not None and needs[i] is not None:
@@ -97,27 +106,34 @@ class DecoderModel:
         """Scores [n_want, vocab] float32 at rows ``want_rows`` (all rows if None)."""
         rt = self.rt
         residual = torch.empty((ctx.rows, self.spec.hidden_size), dtype=torch.float32, device=rt.device)
-        self.embedding.forward(ctx, residual)
+        self._embed(ctx, cache, residual)
         if self.spec.streams:
             return self._forward_streams(residual, ctx, cache, want_rows, n_want)
         if self.embedding_norm is not None:
             self.embedding_norm.forward(residual.clone(), residual)
-        if self.position is not None:
+        if self.position is not None and not self.position_joined:
             self.position.on_embeddings(residual, ctx)
         embedded = None
         if any(j.needs_embedding for j in self.junctions):
             # The embedding's output is read again later: a second gather keeps it (the stream itself moves on).
             embedded = torch.empty_like(residual)
-            self.embedding.forward(ctx, embedded)
+            self._embed(ctx, cache, embedded)
         for i, run in enumerate(self.spec.schedule):
             if run.enter is not None:
                 self.junctions[run.enter[0]].forward(residual, embedded, ctx, run.enter[1])
+            ctx.hand_over = self.hand_over[i]
             self.blocks[run.layer].forward(residual, ctx, cache.memory(i), rt)
             if self.after_run is not None and not ctx.extras.get("graph"):
                 self.after_run(i, residual)
         h = torch.empty((n_want, self.spec.hidden_size), dtype=rt.dtype, device=rt.device)
         self.final_norm.forward(residual, h, want_rows)
         return self._scores(h)
+
+    def _embed(self, ctx: StepContext, cache, out: torch.Tensor) -> None:
+        if self.embedding.cache_need() is None:
+            self.embedding.forward(ctx, out)
+        else:
+            self.embedding.forward(ctx, out, mem=cache.memory(len(self.spec.schedule)))
 
     def _scores(self, h: torch.Tensor) -> torch.Tensor:
         scores = torch.empty((h.shape[0], self.spec.vocab_size), dtype=torch.float32, device=self.rt.device)

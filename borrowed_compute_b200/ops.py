@@ -95,6 +95,20 @@ def _sink_values(sink: Optional[torch.Tensor], heads: int, who: str) -> None:
             raise KernelError(f"{who}: {sink.numel()} sink values for {heads} heads")
 
 
+BIAS_FRONT, BIAS_BACK = 64, 128     # entries of a table of biases ahead of the distance 0 and behind its reach (csrc/common.cuh)
+
+
+def _bias_reach(bias: Optional[torch.Tensor], heads: int, kv_heads: int, who: str) -> int:
+    """The distances a table of biases [kv heads, BIAS_FRONT + reach + BIAS_BACK, heads a kv head] tells apart (0 without a table)."""
+    if bias is None:
+        return 0
+    _need(bias, "bias", torch.float32)
+    reach = bias.shape[1] - BIAS_FRONT - BIAS_BACK if bias.dim() == 3 else 0
+    if reach < 1 or bias.shape[0] != kv_heads or bias.shape[2] != heads // kv_heads:
+        raise KernelError(f"{who}: a table of biases {tuple(bias.shape)} does not fit {heads} heads on {kv_heads}")
+    return reach
+
+
 def _suffix(dtype: torch.dtype) -> str:
     if dtype == torch.float32:
         return "f32"
@@ -150,7 +164,7 @@ _KERNELS_PER_CALL = {"bc_argmax": 2, "bc_moe_plan": 3, "bc_moe_route_f32": 2, "b
 timeline: Optional[list] = None
 label = ""
 _CLASS_OF = {
-    "bc_embed": "embedding", "bc_rmsnorm": "norm", "bc_swiglu": "activation", "bc_rope_append": "rotary + append",
+    "bc_embed": "embedding", "bc_embed_sum": "embedding", "bc_enter_plain": "norm", "bc_rmsnorm": "norm", "bc_swiglu": "activation", "bc_rope_append": "rotary + append",
     "bc_attention_rows": "attention", "bc_attention_decode": "attention", "bc_attention_prefill": "attention",
     "bc_short_conv": "short convolution", "bc_norm_pair": "norm", "bc_delta_split": "low-rank split", "bc_delta": "delta rule",
     "bc_hyper": "streams + norm", "bc_diff": "attention", "bc_polynorm": "activation", "bc_qkv_prepare": "rotary + append",
@@ -208,6 +222,43 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, scale: f
         raise KernelError(f"embed: out is {tuple(out.shape)}, wanted {(rows, E)}")
     _bounds("embed: tokens", tokens, V)
     _call(_fn("bc_embed_" + _suffix(table.dtype)), _ptr(table), _ptr(tokens), _ptr(out), _c_int(rows), _c_int(E), _c_int(V), _c_float(scale), _stream())
+
+
+def embed_sum(table: Optional[torch.Tensor], tokens: torch.Tensor, row_pos: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor, scale: float = 1.0,
+              pairs: Optional[torch.Tensor] = None, mul_prev: int = 0, mul_cur: int = 0, page_table: Optional[torch.Tensor] = None,
+              history: Optional[torch.Tensor] = None, frequencies: Optional[torch.Tensor] = None) -> None:
+    """out[r, :] = table[token] * scale + pairs[b] + s(position), each where it is given (no table: added to what ``out`` holds).
+    ``pairs`` [buckets + 1, E]: b = (token before * mul_prev + token * mul_cur) mod buckets, the last row at position 0; the token
+    before comes from the row ahead or from ``history`` ([pages, 1, 64, 1] int32 behind ``page_table``), where every row leaves its own.
+    ``frequencies`` [ceil(E / 2)] float64: s holds the sine of position * frequency i at 2i and the cosine at 2i + 1."""
+    kind = table if table is not None else pairs
+    for t, name in ((table, "table"), (pairs, "pairs")):
+        if t is not None:
+            _need(t, name, kind.dtype)
+    for t, name in ((tokens, "tokens"), (row_pos, "row_pos"), (row_slot, "row_slot")):
+        _need(t, name, torch.int32)
+    _need(out, "out", torch.float32)
+    rows, E = out.shape
+    if tokens.numel() < rows or row_pos.numel() < rows or row_slot.numel() < rows or (table is not None and table.shape[1] != E):
+        raise KernelError(f"embed_sum: out is {tuple(out.shape)}, tokens {tokens.numel()}")
+    V = table.shape[0] if table is not None else 1
+    if table is not None:
+        _bounds("embed_sum: tokens", tokens, V, rows)
+    buckets = max_pages = n_pages = 0
+    if pairs is not None:
+        _need(page_table, "page_table", torch.int32)
+        _need(history, "history", torch.int32)
+        buckets, max_pages, n_pages = pairs.shape[0] - 1, page_table.shape[1], history.shape[0]
+        if pairs.shape[1] != E or buckets < 1 or tuple(history.shape[1:]) != (1, PAGE, 1):
+            raise KernelError(f"embed_sum: pairs {tuple(pairs.shape)}, history {tuple(history.shape)} do not fit rows of {E}")
+        _bounds_paged("embed_sum", rows, row_pos, row_slot, page_table, n_pages)
+    if frequencies is not None:
+        _need(frequencies, "frequencies", torch.float64)
+        if frequencies.numel() != (E + 1) // 2:
+            raise KernelError(f"embed_sum: {frequencies.numel()} frequencies for rows of {E}")
+    _call(_fn("bc_embed_sum_" + ("f32" if kind is None else _suffix(kind.dtype))), _ptr(table), _ptr(tokens), _c_int(V), _c_float(scale), _ptr(pairs), _c_int(buckets), ctypes.c_longlong(mul_prev),
+          ctypes.c_longlong(mul_cur), _ptr(row_pos), _ptr(row_slot), _ptr(page_table), _c_int(max_pages), _c_int(n_pages), _ptr(history), _ptr(frequencies),
+          _ptr(out), _c_int(rows), _c_int(E), _stream())
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float, gather: Optional[torch.Tensor] = None) -> None:
@@ -578,9 +629,10 @@ def attention_prefill_tc_status(reset: bool = True) -> int:
 def attention_rows(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                    row_pos: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                    window: int = 0, scale: Optional[float] = None, value_dim: Optional[int] = None, chunk: int = 0, sink: bool = False,
-                   out_scale: float = 1.0) -> None:
+                   out_scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every row against its slot's cached positions, one warp a (row, head).
     ``sink`` adds one to the softmax's denominator (a position of score 0 without a value); ``out_scale`` multiplies the result.
+    ``bias``: biases by distance (``parts/distance_bias.py``), in plain units, added to the scores.
     ``value_dim`` (default: ``head_dim``) is the width of a head's values, ``chunk`` > 0 lets a
     position see only those of its own chunk of that many positions, counted from position 0."""
     _need(q, "q")
@@ -603,7 +655,7 @@ def attention_rows(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_cach
     _call(_fn("bc_attention_rows_sink_" + _suffix(q.dtype)), _ptr(q), _c_int(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(page_table),
           _ptr(row_pos), _ptr(row_slot), _ptr(out), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim),
           _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_int(chunk), _c_float(scale), _c_int(1 if sink else 0),
-          _c_float(out_scale), _stream())
+          _c_float(out_scale), _ptr(bias), _c_int(_bias_reach(bias, heads, kv_heads, "attention_rows")), _stream())
 
 
 # ------------------------------------------------------- parts of other mixers and feed-forwards
@@ -796,12 +848,13 @@ def qkv_prepare(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_weight: Optio
 def qkv_prepare_heads(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], cos_sin: Optional[torch.Tensor],
                       row_pos: torch.Tensor, row_slot: torch.Tensor, page_table: torch.Tensor, q_out: torch.Tensor, k_cache: Optional[torch.Tensor],
                       v_cache: Optional[torch.Tensor], heads: int, kv_heads: int, head_dim: int, value_dim: int, rot_dims: int, pairing: int, eps: float,
-                      write_cache: bool = True, value_heads: Optional[int] = None) -> None:
+                      write_cache: bool = True, value_heads: Optional[int] = None, temperature: Optional[Tuple[float, int]] = None) -> None:
     """Between the fused projection (float32) and attention for models that normalise every head by itself: an RMS norm of each
     head of q and of k over its ``head_dim`` values with weights of that many values shared by the heads (when given), rotation of
     the first ``rot_dims`` dimensions of each head (``pairing`` 0: i with i + rot_dims/2; 1: 2i with 2i + 1), q into ``q_out`` and
     k, v into the rows' places in the paged cache.  ``value_heads`` (default: ``kv_heads``) heads of values follow the keys;
-    ``kv_heads`` 0: the projection holds queries alone and nothing is cached."""
+    ``kv_heads`` 0: the projection holds queries alone and nothing is cached.  ``temperature`` = (coef, every): queries at position p
+    are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
     value_heads = kv_heads if value_heads is None else int(value_heads)
     _need(qkv, "qkv", torch.float32)
     _need(q_out, "q_out")
@@ -839,7 +892,8 @@ def qkv_prepare_heads(qkv: torch.Tensor, q_weight: Optional[torch.Tensor], k_wei
           _c_int(n_positions), _ptr(row_pos), _ptr(row_slot), _ptr(page_table), _c_int(page_table.shape[1]), _c_int(n_pages),
           _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(value_heads), _c_int(head_dim),
           _c_int(value_dim), _c_int(rot_dims if n_positions else 0), _c_int(pairing), _c_float(eps), _c_int(0 if q_weight is None else 1),
-          _c_int(1 if write_cache and kv_heads > 0 else 0), _stream())
+          _c_int(1 if write_cache and kv_heads > 0 else 0), _c_float(temperature[0] if temperature else 0.0), _c_int(temperature[1] if temperature else 0),
+          _stream())
 
 
 # ----------------------------------------------------------- recurrences with a decaying outer-product state
@@ -1291,10 +1345,13 @@ def talk_tiles_splits(seqs: int, heads: int, reach: int, window: int, keep_first
 # ------------------------------------------------------------------------------ routed experts
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, row_slot: Optional[torch.Tensor], logits: torch.Tensor, choice: torch.Tensor,
-              weight: torch.Tensor, softmax: bool = False, renorm: bool = False, factor: float = 1.0) -> None:
+              weight: torch.Tensor, softmax: bool = False, renorm: bool = False, factor: float = 1.0, correction: Optional[torch.Tensor] = None,
+              groups: int = 1, keep: int = 1) -> None:
     """choice [rows, top] (int32), weight [rows, top] (float32): every row's ``top`` experts by score, the lower index winning a tie.
     Scores are sigmoid(router @ h) (or a softmax over the experts), computed in float32; weights are the chosen scores, divided by
-    their sum with ``renorm``, then times ``factor``.  Rows whose slot is negative choose nothing (-1).  ``logits`` [rows, experts] float32 receives router @ h."""
+    their sum with ``renorm``, then times ``factor``.  Rows whose slot is negative choose nothing (-1).  ``logits`` [rows, experts] float32 receives router @ h.
+    ``correction`` [experts] is added to the scores for the choice alone; with ``groups`` of neighbouring experts a row chooses within the
+    ``keep`` groups whose largest choice scores are the largest."""
     _need(h, "h")
     _need(router, "router", torch.float32)
     _need(logits, "logits", torch.float32)
@@ -1306,8 +1363,13 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, row_slot: Optional[torch.Te
         raise KernelError(f"moe_route: h {tuple(h.shape)}, router {tuple(router.shape)}, choice {tuple(choice.shape)} do not fit")
     if row_slot is not None:
         _need(row_slot, "row_slot", torch.int32)
+    if correction is not None:
+        _need(correction, "correction", torch.float32)
+        if correction.numel() != E:
+            raise KernelError(f"moe_route: {correction.numel()} corrections for {E} experts")
     _call(_fn("bc_moe_route_" + _suffix(h.dtype)), _ptr(h), _ptr(router), _ptr(row_slot), _ptr(logits), _ptr(choice), _ptr(weight), _c_int(rows), _c_int(E),
-          _c_int(K), _c_int(top), _c_int(1 if softmax else 0), _c_int(1 if renorm else 0), _c_float(factor), _stream())
+          _c_int(K), _c_int(top), _c_int(1 if softmax else 0), _c_int(1 if renorm else 0), _c_float(factor), _ptr(correction), _c_int(groups), _c_int(keep),
+          _stream())
 
 
 def moe_simt_tile_rows() -> int:
@@ -1360,10 +1422,10 @@ def gemm_tc_grouped_accepts(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, table: torch.Tensor, gated: bool, tile_rows: int, max_tiles: int,
-                    relu2: bool = False) -> None:
+                    relu2: bool = False, glu: Optional[Tuple[float, float]] = None) -> None:
     """Rows of x [rows, K] sorted by the matrix they meet, times that matrix of w [matrices, N, K] (``gated``: [matrices, 2 N, K],
     gate rows then up rows, and out = silu(gate) * up in bf16; ``relu2``: out = max(sum, 0)^2 in bf16; else out float32 [rows, N]),
-    on the tcgen05 tensor cores.  ``table``
+    on the tcgen05 tensor cores.  ``glu`` = (limit, alpha): the bounded gate of ``gemm_tc`` for a gated product.  ``table``
     ([0]: tiles; then matrix, first row, rows a tile of at most ``tile_rows``) comes from ``moe_plan`` with the same ``tile_rows``."""
     _need(x, "x", torch.bfloat16)
     _need(w, "w", torch.bfloat16)
@@ -1377,14 +1439,15 @@ def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, table: 
     if kw != K or tuple(out.shape) != (rows, N) or tile_rows not in GROUPED_TILE_ROWS or table.numel() < 1 + 3 * max_tiles:
         raise KernelError(f"gemm_tc_grouped: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}, tiles of {tile_rows} do not fit")
     _call(_fn("bc_gemm_tc_grouped_bf16"), _ptr(x), _ptr(w), _ptr(out), _ptr(table), _c_int(rows), _c_int(matrices), _c_int(N), _c_int(K),
-          _c_int(1 if gated else 2 if relu2 else 0), _c_int(tile_rows), _c_int(max_tiles), _stream())
+          _c_int(1 if gated else 2 if relu2 else 0), _c_int(tile_rows), _c_int(max_tiles), _c_float(glu[0] if glu else 0.0), _c_float(glu[1] if glu else 0.0),
+          _stream())
 
 
 def moe_product(gated: bool, x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, perm: torch.Tensor, weight: torch.Tensor, out: torch.Tensor,
-                top: int, weight_on_input: bool = False) -> None:
+                top: int, weight_on_input: bool = False, glu: Optional[Tuple[float, float]] = None) -> None:
     """The experts' products over rows sorted by expert.  ``gated``: x [rows, K], w [E, 2 N, K] (gate rows, then up rows), out
     [pairs, N] = silu(s g) * (s u) in x's type, s the pair's weight (1 unless ``weight_on_input``).  Else: x [pairs, K] in sorted
-    order, w [E, N, K], out [pairs, N] float32."""
+    order, w [E, N, K], out [pairs, N] float32.  ``glu`` = (limit, alpha): the gated product with the bounded gate of ``gemm_tc``."""
     _need(x, "x")
     _need(w, "w", x.dtype)
     _need(out, "out", x.dtype if gated else torch.float32)
@@ -1394,7 +1457,8 @@ def moe_product(gated: bool, x: torch.Tensor, w: torch.Tensor, table: torch.Tens
     if x.shape[1] != K or out.shape[1] != N or (not gated and x.shape[0] != pairs) or perm.numel() < pairs:
         raise KernelError(f"moe_product: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} do not fit")
     _call(_fn("bc_moe_product_" + _suffix(x.dtype)), _c_int(1 if gated else 0), _ptr(x), _ptr(w), _ptr(table), _ptr(perm), _ptr(weight), _ptr(out),
-          _c_int(pairs), _c_int(E), _c_int(N), _c_int(K), _c_int(top), _c_int(1 if weight_on_input else 0), _stream())
+          _c_int(pairs), _c_int(E), _c_int(N), _c_int(K), _c_int(top), _c_int(1 if weight_on_input else 0), _c_float(glu[0] if glu else 0.0),
+          _c_float(glu[1] if glu else 0.0), _stream())
 
 
 def moe_combine(y: torch.Tensor, choice: torch.Tensor, place: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor,
@@ -1407,6 +1471,20 @@ def moe_combine(y: torch.Tensor, choice: torch.Tensor, place: torch.Tensor, weig
         raise KernelError(f"moe_combine: y {tuple(y.shape)} and residual {tuple(residual.shape)} do not fit")
     _call(_fn("bc_moe_combine"), _ptr(y), _ptr(choice), _ptr(place), _ptr(weight), _ptr(residual), _c_int(rows), _c_int(residual.shape[1]),
           _c_int(top), _c_int(1 if weight_on_output else 0), _stream())
+
+
+def moe_combine_identity(y: torch.Tensor, choice: torch.Tensor, place: torch.Tensor, weight: torch.Tensor, h: torch.Tensor, residual: torch.Tensor,
+                         experts: int) -> None:
+    """``moe_combine`` with the weights on the output, where a choice from ``experts`` on is an identity expert, whose result is the row of ``h`` itself."""
+    _need(y, "y", torch.float32)
+    _need(h, "h")
+    _need(residual, "residual", torch.float32)
+    rows, top = choice.shape
+    width = residual.shape[1]
+    if y.shape[1] != width or residual.shape[0] < rows or h.shape[0] < rows or h.shape[1] != width:
+        raise KernelError(f"moe_combine_identity: y {tuple(y.shape)}, h {tuple(h.shape)} and residual {tuple(residual.shape)} do not fit")
+    _call(_fn("bc_moe_combine_identity_" + _suffix(h.dtype)), _ptr(y), _ptr(choice), _ptr(place), _ptr(weight), _ptr(residual), _ptr(h), _c_int(rows),
+          _c_int(width), _c_int(top), _c_int(experts), _stream())
 
 
 # ---------------------------------------------------------------------------- latent attention
@@ -1649,21 +1727,34 @@ def norm_add(y: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor, eps:
     _call(_fn("bc_norm_add_f32"), _ptr(y), _ptr(weight), _ptr(residual), _c_int(rows), _c_int(E), _c_float(eps), _stream())
 
 
-def norm_add_norm(y: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor, eps: float, next_weight: torch.Tensor, out: torch.Tensor,
+def norm_add_norm(y: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor, eps: float, next_weight: Optional[torch.Tensor], out: torch.Tensor,
                   next_eps: float) -> None:
     """norm_add, then out[r] = residual[r] * rsqrt(mean(residual[r]^2) + next_eps) * next_weight in out's type, and y = 0: what lies
-    between the two sublayers of a block that norms before and after each, in one kernel.  y, residual and the weights float32."""
+    between the two sublayers of a block that norms before and after each, in one kernel.  y, residual and the weights float32.
+    ``next_weight`` None: the next sublayer reads the stream itself, out = residual in out's type."""
     _need(y, "y", torch.float32)
     _need(weight, "weight", torch.float32)
-    _need(next_weight, "next_weight", torch.float32)
+    if next_weight is not None:
+        _need(next_weight, "next_weight", torch.float32)
     _need(residual, "residual", torch.float32)
     _need(out, "out")
     rows, E = y.shape
-    if residual.shape[0] < rows or residual.shape[1] != E or weight.numel() != E or next_weight.numel() != E or tuple(out.shape) != (rows, E):
-        raise KernelError(f"norm_add_norm: y {tuple(y.shape)}, residual {tuple(residual.shape)}, out {tuple(out.shape)}, weights {weight.numel()} and "
-                          f"{next_weight.numel()} do not fit")
+    if residual.shape[0] < rows or residual.shape[1] != E or weight.numel() != E or (next_weight is not None and next_weight.numel() != E) \
+            or tuple(out.shape) != (rows, E):
+        raise KernelError(f"norm_add_norm: y {tuple(y.shape)}, residual {tuple(residual.shape)}, out {tuple(out.shape)} and the weights do not fit")
     _call(_fn("bc_norm_add_norm_" + _suffix(out.dtype)), _ptr(y), _ptr(weight), _ptr(residual), _ptr(next_weight), _ptr(out), _c_int(rows), _c_int(E),
           _c_float(eps), _c_float(next_eps), _stream())
+
+
+def enter_plain(residual: torch.Tensor, out: torch.Tensor, y: torch.Tensor) -> None:
+    """out = residual in out's type and y = 0: ahead of a sublayer that reads the stream itself and adds its result into y."""
+    _need(residual, "residual", torch.float32)
+    _need(y, "y", torch.float32)
+    _need(out, "out")
+    rows, E = residual.shape
+    if tuple(out.shape) != (rows, E) or tuple(y.shape) != (rows, E):
+        raise KernelError(f"enter_plain: residual {tuple(residual.shape)}, out {tuple(out.shape)} and y {tuple(y.shape)} differ")
+    _call(_fn("bc_enter_plain_" + _suffix(out.dtype)), _ptr(residual), _ptr(out), _ptr(y), _c_int(rows), _c_int(E), _stream())
 
 
 def relu2(z: torch.Tensor, out: torch.Tensor) -> None:
@@ -1818,7 +1909,7 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
                      row_pos: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                      window: int = 0, scale: Optional[float] = None, splits: Optional[int] = None, fuse: int = 0,
                      cos_sin: Optional[torch.Tensor] = None, pairing: int = 0, via_scratch: bool = False,
-                     reach: Optional[int] = None, sink: bool = False, out_scale: float = 1.0) -> None:
+                     reach: Optional[int] = None, sink: bool = False, out_scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """Attention of one new row a sequence (bf16): the cached positions are split across
     blocks and the heads of a kv head share each read; results are merged in a fixed order.
     Two to eight splits form a thread-block cluster and merge through one another's shared
@@ -1828,8 +1919,8 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
     value are appended to the cache first (what rope_append would have done).  ``reach``:
     a bound on the positions any row reaches (else what the page table can hold); the
     number of splits is chosen by it, no result depends on it.  ``sink`` adds one to the softmax's
-    denominator (a position of score 0 without a value), ``out_scale`` multiplies the result: both
-    with the plain kernel (``fuse`` 0) only."""
+    denominator (a position of score 0 without a value), ``out_scale`` multiplies the result, ``bias``
+    (biases by distance, ``parts/distance_bias.py``, in log2 units) is added to the scores: all three with the plain kernel (``fuse`` 0) only."""
     _need(q, "q", torch.bfloat16)
     _need(k_cache, "k_cache", torch.bfloat16)
     _need(v_cache, "v_cache", torch.bfloat16)
@@ -1861,13 +1952,14 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
         if bounds_check and not torch.cuda.is_current_stream_capturing():
             _bounds("attention_decode: row_pos (against the rotary table)", row_pos.reshape(-1)[:rows][row_slot.reshape(-1)[:rows] >= 0], cos_sin.shape[0])
     _bounds_paged("attention_decode", rows, row_pos, row_slot, page_table, k_cache.shape[0])
-    if sink or out_scale != 1.0:
+    if sink or out_scale != 1.0 or bias is not None:
         if fuse != 0:
-            raise KernelError("attention_decode: a sink or a factor comes with the plain kernel (fuse 0)")
+            raise KernelError("attention_decode: a sink, biases or a factor comes with the plain kernel (fuse 0)")
         _call(_fn("bc_attention_decode_sink_bf16"), _ptr(q), _c_int(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(row_pos),
               _ptr(row_slot), _ptr(out), _ptr(scratch), _ptr(counters), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
               _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_float(scale), _c_int(splits),
-              _c_int(4 if via_scratch else 0), _c_int(1 if sink else 0), _c_float(out_scale), _stream())
+              _c_int(4 if via_scratch else 0), _c_int(1 if sink else 0), _c_float(out_scale), _ptr(bias),
+              _c_int(_bias_reach(bias, heads, kv_heads, "attention_decode")), _stream())
         return
     _call(_fn("bc_attention_decode_fused_bf16"), _ptr(q), _c_int(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(row_pos),
           _ptr(row_slot), _ptr(out), _ptr(scratch), _ptr(counters), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
@@ -1891,12 +1983,12 @@ def attention_tiles_accepts(heads: int, kv_heads: int, head_dim: int, value_dim:
 def attention_tiles(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_cache: torch.Tensor, page_table: torch.Tensor,
                     seq_rows: torch.Tensor, seq_slot: torch.Tensor, seq_start: torch.Tensor, out: torch.Tensor, seqs: int, max_new: int,
                     heads: int, kv_heads: int, head_dim: int, value_dim: int, window: int = 0, chunk: int = 0,
-                    scale: Optional[float] = None, sink: bool = False, out_scale: float = 1.0) -> None:
+                    scale: Optional[float] = None, sink: bool = False, out_scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every sequence's new rows (many, or one) against its cached positions on mma.sync
     tiles, bf16, with values of their own width, a sliding window and/or a chunk mask (``chunk`` > 0: a position
     sees only those of its own chunk of that many positions, counted from position 0).  ``sink`` adds one to the
     softmax's denominator (a position of score 0 without a value), or, given as a float32 tensor [heads], e^sink[head];
-    ``out_scale`` multiplies the result."""
+    ``out_scale`` multiplies the result; ``bias``: biases by distance in log2 units."""
     for t, name in ((q, "q"), (k_cache, "k_cache"), (v_cache, "v_cache"), (out, "out")):
         _need(t, name, torch.bfloat16)
     if isinstance(sink, torch.Tensor):
@@ -1915,7 +2007,8 @@ def attention_tiles(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_cac
     _call(_fn("bc_attention_prefill_sink_bf16"), _ptr(q), _c_int(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(seq_rows),
           _ptr(seq_slot), _ptr(seq_start), _ptr(out), _c_int(seqs), _c_int(max_new), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
           _c_int(value_dim), _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_int(chunk), _c_float(scale),
-          _c_int(0 if sink is None or sink is False else 1), _ptr(sink if isinstance(sink, torch.Tensor) else None), _c_float(out_scale), _stream())
+          _c_int(0 if sink is None or sink is False else 1), _ptr(sink if isinstance(sink, torch.Tensor) else None), _c_float(out_scale), _ptr(bias),
+          _c_int(_bias_reach(bias, heads, kv_heads, "attention_tiles")), _stream())
 
 
 def attention_prefill_tc_accepts(heads: int, kv_heads: int, head_dim: int, q: Optional[torch.Tensor] = None, q_stride: int = 0,
@@ -1933,7 +2026,7 @@ def attention_prefill(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_c
                       seq_rows: torch.Tensor, seq_slot: torch.Tensor, seq_start: torch.Tensor, out: torch.Tensor, seqs: int, max_new: int,
                       heads: int, kv_heads: int, head_dim: int, window: int = 0, scale: Optional[float] = None,
                       use_tc: Optional[bool] = None, chunk: int = 0, value_dim: Optional[int] = None, sink: bool = False,
-                      out_scale: float = 1.0) -> None:
+                      out_scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every sequence's new rows against its cached positions (which
     include the new rows' own keys and values), bf16.  Head sizes 64 and 128 run on the
     tcgen05 tensor cores, 128 query rows a block (scores and output accumulate in TMEM);
@@ -1941,7 +2034,7 @@ def attention_prefill(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_c
     ``chunk`` > 0: a position sees only those of its own chunk of that many positions, counted from position 0.
     ``value_dim`` (default ``head_dim``): the width of a head's values, in v_cache and in out.
     ``sink`` adds one to the softmax's denominator (a position of score 0 without a value), or, given as a float32 tensor [heads],
-    e^sink[head]; ``out_scale`` multiplies the result."""
+    e^sink[head]; ``out_scale`` multiplies the result; ``bias``: biases by distance (``parts/distance_bias.py``) in log2 units."""
     value_dim = head_dim if value_dim is None else int(value_dim)
     if isinstance(sink, torch.Tensor):
         _sink_values(sink, heads, "attention_prefill")
@@ -1976,11 +2069,11 @@ def attention_prefill(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_c
               _ptr(seq_rows), _ptr(seq_slot), _ptr(seq_start), _ptr(out), _c_int(seqs), _c_int(max_new), _c_int(heads), _c_int(kv_heads),
               _c_int(head_dim), _c_int(value_dim), _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_int(chunk),
               _c_float(scale), _c_int(0 if sink is None or sink is False else 1), _ptr(sink if isinstance(sink, torch.Tensor) else None),
-              _c_float(out_scale), _stream())
+              _c_float(out_scale), _ptr(bias), _c_int(_bias_reach(bias, heads, kv_heads, "attention_prefill")), _stream())
         return
-    if chunk > 0 or value_dim != head_dim or (sink is not None and sink is not False) or out_scale != 1.0:
+    if chunk > 0 or value_dim != head_dim or (sink is not None and sink is not False) or out_scale != 1.0 or bias is not None:
         attention_tiles(q, q_stride, k_cache, v_cache, page_table, seq_rows, seq_slot, seq_start, out, seqs, max_new, heads, kv_heads, head_dim,
-                        value_dim, window=window, chunk=chunk, scale=scale, sink=sink, out_scale=out_scale)
+                        value_dim, window=window, chunk=chunk, scale=scale, sink=sink, out_scale=out_scale, bias=bias)
         return
     _call(_fn("bc_attention_prefill_bf16"), _ptr(q), _c_int(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(seq_rows),
           _ptr(seq_slot), _ptr(seq_start), _ptr(out), _c_int(seqs), _c_int(max_new), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),

@@ -187,12 +187,14 @@ class CacheNeed:
     latest positions are ever read; ``chunk`` > 0 if a position only ever reads those of its
     own chunk of that many positions (counted from position 0), so that whole chunks behind
     the newest one can be let go.  ``keep_first`` > 0 if the first that many positions of a sequence stay readable
-    whatever the window (they are never let go).  Runs with equal needs share one storage group."""
+    whatever the window (they are never let go).  ``dtype`` None keeps values of the compute type; another type is kept as it is (an
+    embedding that looks back at token ids asks for int32).  Runs with equal needs share one storage group."""
 
     planes: Tuple[Tuple[int, int], ...]
     window: int = 0
     chunk: int = 0
     keep_first: int = 0
+    dtype: Optional[torch.dtype] = None
 
     def __post_init__(self):
         self.planes = tuple((int(h), int(w)) for h, w in self.planes)
@@ -207,14 +209,14 @@ class CacheNeed:
         return CacheNeed(((kv_heads, head_dim), (kv_heads, head_dim if value_dim is None else value_dim)), window, chunk, keep_first)
 
     def key(self) -> Tuple:
-        return (self.planes, self.window, self.chunk, self.keep_first)
+        return (self.planes, self.window, self.chunk, self.keep_first, self.dtype)
 
     def widened(self, other: "CacheNeed") -> "CacheNeed":
         """What serves this need and ``other`` (of a run that reads the same memory) alike: every position either of them reads is kept."""
-        if self.planes != other.planes:
+        if self.planes != other.planes or self.dtype != other.dtype:
             raise ValueError(f"a run cannot read planes {other.planes} out of memory with planes {self.planes}")
         return CacheNeed(self.planes, window=max(self.window, other.window) if self.window and other.window else 0,
-                         chunk=self.chunk if self.chunk == other.chunk else 0, keep_first=max(self.keep_first, other.keep_first))
+                         chunk=self.chunk if self.chunk == other.chunk else 0, keep_first=max(self.keep_first, other.keep_first), dtype=self.dtype)
 
     def values_per_token(self) -> int:
         return sum(h * w for h, w in self.planes)
@@ -275,6 +277,10 @@ class StepContext:
     host_seq_slot: Tuple[int, ...] = ()
     host_seq_start: Tuple[int, ...] = ()
     extras: Dict[str, Any] = field(default_factory=dict)
+    # Between two blocks that read the stream itself (Block.enters_plain) with nothing in between: the model sets ``hand_over``
+    # for the first, which then leaves the stream in the activation type and a cleared float buffer in ``handed`` for the second.
+    hand_over: bool = False
+    handed: Optional[Tuple[torch.Tensor, torch.Tensor]] = None
 
 
 # ------------------------------------------------------------------------------- interfaces
@@ -384,9 +390,19 @@ class FeedForward(Part):
 
 
 class Embedding(Part):
-    def forward(self, ctx: StepContext, residual: torch.Tensor) -> None:
+    """An embedding that asks for token-indexed memory (``cache_need``) finds it in ``mem`` at every call; one that does not is called
+    without ``mem``."""
+
+    def forward(self, ctx: StepContext, residual: torch.Tensor, mem: Optional[RunMemory] = None) -> None:
         """residual[r] = embedding of ctx.tokens[r], as float32."""
         raise NotImplementedError
+
+    def cache_need(self) -> Optional[CacheNeed]:
+        return None
+
+    def join(self, position: PositionEncoding) -> bool:
+        """True if this embedding adds what ``position.on_embeddings`` would, from now on: the model then leaves that call out."""
+        return False
 
     def table(self) -> Optional[torch.Tensor]:
         """The [vocab, hidden] table, for a head tied to it."""
@@ -407,6 +423,8 @@ class Block(Part):
 
     # True for blocks whose forward takes a StreamBundle instead of one residual tensor (ModelSpec.streams > 0).
     STREAMS = False
+    # True for a block whose first sublayer reads the residual stream itself, rounded to the activation type (no norm ahead of it).
+    enters_plain = False
     ROLES: Dict[str, Registry] = {}
     OPTIONAL: Tuple[str, ...] = ()
 

@@ -10,7 +10,8 @@ without a norm of its own reads what the mixer reads, x += mixer(h) + feed_forwa
 h = norm1(x).
 
 The sandwich block: a norm before and after each sublayer, x += norm1b(mixer(conv(norm1(x)))); x += norm2b(ff(norm2(x))).
-The second half may be left out, and so may the short convolution (or token shift) of the mixer's input.
+The second half may be left out, and so may the short convolution (or token shift) of the mixer's input.  So may the norms ahead of
+the sublayers, which then read x itself: x += norm1b(mixer(x)); x += norm2b(ff(x)).
 
 The hyper-connected block: a pre-norm block on a bundle of streams (``parts/streams.py``), each sublayer between the two ends of its
 connection, its result scaled channel by channel.  The feed-forward and what belongs to it may be left out, and so may the scales."""
@@ -98,11 +99,14 @@ class SandwichBlock(Block):
     itself: the sublayer adds into a cleared float buffer, and one kernel norms that and adds it."""
 
     ROLES = {"norm1": NORMS, "conv": CONVOLUTIONS, "mixer": MIXERS, "norm1b": NORMS, "norm2": NORMS, "feed_forward": FEED_FORWARDS, "norm2b": NORMS}
-    OPTIONAL = ("conv", "norm2", "feed_forward", "norm2b")
+    OPTIONAL = ("norm1", "conv", "norm2", "feed_forward", "norm2b")
 
     def __init__(self, parts, hidden_size: int):
         super().__init__(parts, hidden_size)
-        if len({self.norm2 is None, self.feed_forward is None, self.norm2b is None}) != 1:
+        self.enters_plain = self.norm1 is None
+        if self.enters_plain and (self.conv is not None or self.norm2 is not None):
+            raise ValueError("a sandwich block whose mixer reads the stream itself has no convolution and no norm ahead of its feed-forward")
+        if len({self.feed_forward is None, self.norm2b is None} | (set() if self.enters_plain else {self.norm2 is None})) != 1:
             raise ValueError("a sandwich block has a feed-forward with both of its norms, or none of the three")
         for role in ("norm1b", "norm2b"):
             if getattr(self, role) is not None and type(getattr(self, role)) is not RMSNorm:
@@ -117,6 +121,9 @@ class SandwichBlock(Block):
 
     def forward(self, residual: torch.Tensor, ctx: StepContext, mem: RunMemory, rt: Runtime) -> None:
         rows = residual.shape[0]
+        if self.enters_plain:
+            self._forward_plain(residual, ctx, mem, rt)
+            return
         h = torch.empty((rows, self.hidden_size), dtype=rt.dtype, device=residual.device)
         y = torch.zeros((rows, self.hidden_size), dtype=torch.float32, device=residual.device)
         if self.conv is not None and ctx.decode and type(self.norm1) is RMSNorm and isinstance(self.conv, CausalConvResidual):
@@ -149,6 +156,29 @@ class SandwichBlock(Block):
                 self.norm2.forward(residual, h)
             self.feed_forward.forward(h, y, ctx)
             ops.norm_add(y, self.norm2b.weight, residual, self.norm2b.eps)
+
+
+    def _forward_plain(self, residual: torch.Tensor, ctx: StepContext, mem: RunMemory, rt: Runtime) -> None:
+        """Without norms ahead of the sublayers: one kernel after each norms its result into the stream, leaves the stream in the
+        activation type for the next sublayer and clears the buffer for that one's result, from layer to layer where the next block
+        is of this kind too (``StepContext.hand_over``)."""
+        if ctx.handed is not None:
+            h, y = ctx.handed
+            ctx.handed = None
+        else:
+            h = torch.empty(residual.shape, dtype=rt.dtype, device=residual.device)
+            y = torch.empty_like(residual)
+            ops.enter_plain(residual, h, y)
+        last = self.norm1b if self.feed_forward is None else self.norm2b
+        self.mixer.forward(h, y, ctx, mem)
+        if self.feed_forward is not None:
+            ops.norm_add_norm(y, self.norm1b.weight, residual, self.norm1b.eps, None, h, self.norm1b.eps)
+            self.feed_forward.forward(h, y, ctx)
+        if ctx.hand_over:
+            ops.norm_add_norm(y, last.weight, residual, last.eps, None, h, last.eps)
+            ctx.handed = (h, y)
+        else:
+            ops.norm_add(y, last.weight, residual, last.eps)
 
 
 @BLOCKS.register("hyper_connected")
