@@ -521,15 +521,18 @@ def _against(costs, measured, pk, fp32_tflops):
     return out
 
 
-def _bench_models(configs, costs_of, vocab, out, pk, rng, fp32_tflops, batch, prompt, steps, warmup):
+def _bench_models(configs, costs_of, vocab, out, pk, rng, fp32_tflops, batch, prompt, steps, warmup, prepare=None):
     """For each (name, config): decode steps of ``batch`` sequences after prompts of ``prompt`` tokens, one prompt alone,
-    all prompts in one step, and every kernel class launch by launch against ``costs_of(name, config)``."""
+    all prompts in one step, and every kernel class launch by launch against ``costs_of(name, config)``.  ``prepare(name, engine)``
+    runs once on every fresh engine."""
     import torch
 
     from borrowed_compute_b200.engine import Engine, StepEntry, StepProfile
 
     for name, cfg in configs.items():
         eng = Engine.from_random(cfg, seed=1, max_tokens=batch * (prompt + 256), max_slots=batch, max_seq=prompt + 256)
+        if prepare is not None:
+            prepare(name, eng)
         prompts = [[int(t) for t in rng.integers(0, vocab, prompt)] for _ in range(batch)]
         # the step of all prompts once untimed (a kernel's first launch loads it), then timed inside timed_decode
         warm = [eng.acquire() for _ in range(batch)]
@@ -1010,6 +1013,124 @@ def bench_duratar(pk, rng, size="wide", layers=4, batch=8, prompt=PROMPT, steps=
     return _bench_models(configs, costs_of, c["vocab"], out, pk, rng, FP32_TFLOPS, batch, prompt, steps, warmup)
 
 
+# ------------------------------------------------------------------ the seventh architecture
+KODULIX_SIZES = {
+    # the width and heads of the 8B shape; 32 experts of 2,048 of which a row uses 4, beside 8 identity experts, in 4 groups of which 2
+    # are kept, and a shared expert of 4,096; 32 buckets of distances up to 128
+    "wide": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, rows=32, reach=128, experts=32, top=4, identity=8, groups=4, keep=2, ff=2048,
+                 shared=4096, vocab=32000),
+    # a 2,048-wide model: values half as wide as keys, 64 experts of 1,408 of which a row uses 6, distances up to 1,024
+    "mid": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=64, rows=64, reach=1024, experts=64, top=6, identity=16, groups=8, keep=4, ff=1408,
+                shared=2816, vocab=32000),
+}
+
+
+def kodulix_config(width, heads, kv_heads, dim, vdim, rows, reach, experts, top, identity, groups, keep, ff, shared, vocab, layers):
+    """``layers`` layers of the Kodulix design: attention with biases by distance, experts in groups beside identity experts."""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": 1.0 / dim ** 0.5, "bias_rows": rows, "bias_max": reach,
+             "q_temp": {"coef": 0.1, "every": 1024}}
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "shared": {"ff": shared, "limit": 7.0},
+           "router": {"experts": experts, "top": top, "identity": identity, "groups": {"count": groups, "keep": keep}}}
+    return {"architecture": "Kodulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "logit_scale": 1.0,
+            "embedding": {"bigram": {"buckets": vocab, "mul_prev": 31, "mul_cur": 7}}, "layers": [{"type": "attention", "mixer": mixer, "mlp": mlp}] * layers}
+
+
+def kodulix_costs(c, layers, batch, ctx_len, T) -> dict:
+    """What each kernel class of the Kodulix model has to move in a decode step (bytes) and to compute in a prompt step of T tokens
+    (operations, or bytes where it only moves data), summed over the model's layers.  c["counted"] tells how many of a row's choices
+    are experts with matrices, in a decode step and in a prompt, and how many of these experts a decode step touches a layer: counted in
+    steps of the model that is timed, since its random routers favour some experts."""
+    E, H, G, D, DV, V = c["width"], c["heads"], c["kv_heads"], c["dim"], c["vdim"], c["vocab"]
+    X, XI, f, fs, B = c["experts"], c["experts"] + c["identity"], c["ff"], c["shared"], batch
+    n_qkv, top = H * D + G * D + G * DV, c["top"]
+    k, k_prompt, touched = c["counted"]
+    pairs = T * (T + 1) / 2.0
+    decode = {
+        "embedding": B * E * 8.0,
+        # a result read and cleared, the stream read and written, a rounded row written: twice a layer
+        "norm": 2 * layers * (B * E * 18.0 + E * 4.0) + B * E * 6.0,
+        "qkv product": layers * (2.0 * n_qkv * E + B * (2.0 * E + 4.0 * n_qkv)),
+        "rotary + append": layers * B * 6.0 * n_qkv,
+        "attention": layers * B * ((ctx_len + 1) * G * (D + DV) * 2.0 + 2.0 * H * (D + DV)),
+        "output product": layers * (2.0 * H * DV * E + B * (2.0 * H * DV + 8.0 * E)),
+        "routing": layers * (4.0 * XI * E + B * (2.0 * E + 8.0 * top)),
+        "expert sort": layers * B * top * 16.0,
+        "expert gather": layers * B * k * E * 4.0,
+        "expert sum": layers * B * (k * E * 4.0 + E * 10.0),
+        "expert product": layers * (touched * 3.0 * f * E * 2.0 + B * k * (2.0 * E + 4.0 * f + 4.0 * E)),
+        "gate/up product": layers * (4.0 * fs * E + B * (2.0 * E + 2.0 * fs)),
+        "down product": layers * (2.0 * fs * E + B * (2.0 * fs + 8.0 * E)),
+        "head product": 2.0 * V * E + B * (2.0 * E + 4.0 * V),
+    }
+    prefill = {
+        "embedding": ("bytes", T * E * 8.0),
+        "norm": ("bytes", 2 * layers * T * E * 18.0),
+        "qkv product": ("flops", layers * 2.0 * T * n_qkv * E),
+        "rotary + append": ("bytes", layers * T * 6.0 * n_qkv),
+        "attention": ("flops", layers * 2.0 * H * (D + DV) * pairs),
+        "output product": ("flops", layers * 2.0 * T * E * H * DV),
+        "routing": ("flops32", layers * 2.0 * T * XI * E),
+        "expert sort": ("bytes", layers * T * top * 16.0),
+        "expert gather": ("bytes", layers * T * k_prompt * E * 4.0),
+        "expert sum": ("bytes", layers * T * (k_prompt * E * 4.0 + E * 10.0)),
+        "expert product": ("flops", layers * 2.0 * T * k_prompt * 3.0 * f * E),
+        "gate/up product": ("flops", layers * 4.0 * T * fs * E),
+        "down product": ("flops", layers * 2.0 * T * fs * E),
+    }
+    return {"decode": decode, "prefill": prefill}
+
+
+def bench_kodulix(pk, rng, size="wide", layers=4, batch=8, prompt=PROMPT, steps=32, warmup=4) -> dict:
+    """Prompt and decode throughput of a Kodulix model of ``layers`` layers at sizes that resemble a real model's layers (random weights),
+    beside a Pozirax model, the closest of the other designs (attention with normed heads, routed experts plus a shared one), and a Llama
+    model (attention over every earlier position), both of the same width, attention heads, vocabulary and depth; the Pozirax model's
+    experts are as many and as wide, the Llama model's feed-forward as wide as the experts a row uses.  Every kernel class of the three
+    against its own bytes or operations."""
+    c = dict(KODULIX_SIZES[size])
+    same = {k: c[k] for k in ("width", "heads", "kv_heads", "dim", "vdim", "experts", "top", "ff", "shared", "vocab")}
+    z = dict(POZIRAX_SIZES[size], **same)
+    configs = {"kodulix": kodulix_config(layers=layers, **KODULIX_SIZES[size]), "pozirax": pozirax_config(layers=layers, **z),
+               "llama": llama_like(c["width"], c["heads"], c["kv_heads"], c["dim"], c["top"] * c["ff"] + c["shared"], c["vocab"], layers)}
+    out = {"size": size, "sizes": KODULIX_SIZES[size], "beside": z, "layers": layers, "batch": batch, "prompt": prompt,
+           "between": "weights of a step exceed the L2", "peaks": pk, "fp32_cuda_core_tflops_nominal": round(FP32_TFLOPS, 1)}
+
+    def prepare(name, eng):
+        """Embedded rows as large as the sinusoids beside them (else every row routes alike), and a count of what the experts get."""
+        if name != "kodulix":
+            return
+        from borrowed_compute_b200 import ops
+        from borrowed_compute_b200.engine import StepEntry
+
+        eng.model.embedding.weight.mul_(50.0)
+        chosen, plain = [], ops.moe_combine_identity
+        ops.moe_combine_identity = lambda y, choice, *rest: (chosen.append(choice.cpu().numpy()), plain(y, choice, *rest))
+        eng.use_graphs = False
+        slots = [eng.acquire() for _ in range(batch)]
+        for _ in range(2):
+            chosen.clear()
+            tokens = [[int(t) for t in rng.integers(0, c["vocab"], 64)] for _ in slots]
+            eng.step([StepEntry(s, t, want=()) for s, t in zip(slots, tokens)])
+            k_prompt = sum((x < c["experts"]).sum() / x.shape[0] for x in chosen) / len(chosen)
+        k, touched, reps = 0.0, 0.0, 8
+        for _ in range(reps):
+            chosen.clear()
+            eng.step([StepEntry(s, (int(rng.integers(0, c["vocab"])),), want=(0,)) for s in slots])
+            k += sum((x < c["experts"]).sum() / x.shape[0] for x in chosen) / len(chosen) / reps
+            touched += sum(len(set(x[x < c["experts"]].tolist())) for x in chosen) / len(chosen) / reps
+        for s in slots:
+            eng.release(s)
+        ops.moe_combine_identity, eng.use_graphs = plain, True
+        c["counted"] = (float(k), float(k_prompt), float(touched))
+        out["counted"] = {"experts_a_row": round(float(k), 2), "experts_a_row_prompt": round(float(k_prompt), 2), "experts_touched_a_step": round(float(touched), 2)}
+
+    def costs_of(name, cfg):
+        if name == "llama":
+            return class_costs(cfg, layers, batch, batch * (prompt + 2), prompt)
+        return (kodulix_costs if name == "kodulix" else pozirax_costs)(c if name == "kodulix" else z, layers, batch, prompt + 2, prompt)
+
+    return _bench_models(configs, costs_of, c["vocab"], out, pk, rng, FP32_TFLOPS, batch, prompt, steps, warmup, prepare)
+
+
 def run_ours(args) -> dict:
     import numpy as np
     import torch
@@ -1168,9 +1289,9 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 and 64 and the two other shapes")
     ap.add_argument("--no-breakdown", action="store_true", help="skip the per-class timing of one decode and one prompt step")
-    ap.add_argument("--point", default="", choices=["", "long", "13b", "3b", "tiny", "fegidra", "pozirax", "fudelorn", "logirax", "duratar"],
+    ap.add_argument("--point", default="", choices=["", "long", "13b", "3b", "tiny", "fegidra", "pozirax", "fudelorn", "logirax", "duratar", "kodulix"],
                     help="run one of the further workloads alone and print its figures (not the default run's one JSON line)")
-    ap.add_argument("--size", default="wide", choices=sorted(FEGIDRA_SIZES), help="with --point fegidra, pozirax, fudelorn, logirax or duratar: which sizes")
+    ap.add_argument("--size", default="wide", choices=sorted(FEGIDRA_SIZES), help="with --point fegidra, pozirax, fudelorn, logirax, duratar or kodulix: which sizes")
     args = ap.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable": "the reference is a Rust workspace (no setup.py or pyproject) "
@@ -1191,7 +1312,8 @@ def main() -> int:
                "pozirax": lambda: bench_pozirax(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
                "fudelorn": lambda: bench_fudelorn(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
                "logirax": lambda: bench_logirax(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
-               "duratar": lambda: bench_duratar(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup)}[args.point]
+               "duratar": lambda: bench_duratar(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup),
+               "kodulix": lambda: bench_kodulix(peaks(), rng, args.size, args.layers or 4, args.batch, args.prompt, min(args.steps, 32), args.warmup)}[args.point]
         print(json.dumps({"point": args.point, **one()}))
         return 0
     print(json.dumps(run_ours(args)))

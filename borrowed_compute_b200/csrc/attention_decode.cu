@@ -56,7 +56,7 @@ extern "C" int bc_attention_decode_set_trace(long long* buf) { return (int)cudaM
 // The four computing warps among themselves (the fifth warp, where there is one, is not part of it).
 __device__ __forceinline__ void ad_workers_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-template <int D, bool TMA, bool BIAS>
+template <int D, int DV, bool TMA, bool BIAS>
 __global__ void __launch_bounds__(TMA ? AD_THREADS_TMA : AD_THREADS)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
                         const int* __restrict__ page_table, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
@@ -64,16 +64,17 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         int n_pages, int window, float scale_log2, const float2* __restrict__ cos_sin, int pairing, int fuse,
                         int k_off, int v_off, bf16* __restrict__ k_write, bf16* __restrict__ v_write, int use_cluster, int sink,
                         float out_scale, const float* __restrict__ bias, int bias_reach) {
-    constexpr int CHUNKS = D / 8;              // 16-byte chunks a row
-    constexpr int TILE_BYTES = 64 * D * 2;     // one page of one kv head
+    constexpr int CHUNKS = D / 8, VCHUNKS = DV / 8;                      // 16-byte chunks a row of keys, of values
+    constexpr int K_BYTES = 64 * D * 2, STAGE_BYTES = 64 * (D + DV) * 2;   // one page of one kv head: its keys, then its values
     constexpr int KD = D / 16;                 // k-steps of Q K^T
-    constexpr int ND = D / 8;                  // 8-wide dimension blocks of the output
+    constexpr int ND = DV / 8;                 // 8-wide dimension blocks of the output
     extern __shared__ __align__(1024) uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);   // TMA's swizzle wants 1024-byte alignment
     __shared__ int is_last;
     __shared__ int page_ids[AD_PAGES_KEPT];   // the pages of this block's first tiles (-1: none)
     __shared__ __align__(8) uint64_t full_bars[AD_STAGES], empty_bars[AD_STAGES];
     auto offset = [](int r, int c) { return TMA ? tma_tile_offset(r, c) : tile_offset<D>(r, c); };
+    auto v_offset = [](int r, int c) { return TMA ? tma_tile_offset(r, c) : tile_offset<DV>(r, c); };
     const uint32_t full0 = smem_u32(&full_bars[0]), empty0 = smem_u32(&empty_bars[0]);
     if (TMA && threadIdx.x == 0) {
         for (int s = 0; s < AD_STAGES; s++) {
@@ -97,7 +98,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     if (slot < 0) {
         pdl_wait();
         if (split == 0)
-            for (int i = threadIdx.x; i < group * D; i += AD_THREADS) out[((size_t)r * H + (size_t)g * group) * D + i] = __float2bfloat16_rn(0.0f);
+            for (int i = threadIdx.x; i < group * DV; i += AD_THREADS) out[((size_t)r * H + (size_t)g * group) * DV + i] = __float2bfloat16_rn(0.0f);
         return;
     }
     const int lo = window > 0 && pos + 1 > window ? pos + 1 - window : 0;
@@ -126,29 +127,33 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     };
     auto load_tile = [&](int tile, int stage) {
         const int page = page_of(tile);
-        const uint32_t kb = ad_smem(smem + (size_t)stage * 2 * TILE_BYTES), vb = kb + TILE_BYTES;
+        const uint32_t kb = ad_smem(smem + (size_t)stage * STAGE_BYTES), vb = kb + K_BYTES;
         if (TMA) {   // called by the asking thread alone
             if (page < 0) {
                 mbar_arrive(full0 + 8 * stage);   // nothing comes: the stage's phase ends at once
                 return;
             }
             const int y = (page * G + g) * BC_PAGE;
-            mbar_expect_tx(full0 + 8 * stage, 2 * TILE_BYTES);
+            mbar_expect_tx(full0 + 8 * stage, STAGE_BYTES);
 #pragma unroll
-            for (int b = 0; b < D / 64; b++) {
-                tma_load_2d(kb + b * 8192, &map_k, full0 + 8 * stage, b * 64, y);
-                tma_load_2d(vb + b * 8192, &map_v, full0 + 8 * stage, b * 64, y);
-            }
+            for (int b = 0; b < D / 64; b++) tma_load_2d(kb + b * 8192, &map_k, full0 + 8 * stage, b * 64, y);
+#pragma unroll
+            for (int b = 0; b < DV / 64; b++) tma_load_2d(vb + b * 8192, &map_v, full0 + 8 * stage, b * 64, y);
             return;
         }
         if (page < 0) return;
         const bf16* ks = k_cache + ((size_t)page * G + g) * BC_PAGE * D;
-        const bf16* vs = v_cache + ((size_t)page * G + g) * BC_PAGE * D;
+        const bf16* vs = v_cache + ((size_t)page * G + g) * BC_PAGE * DV;
         for (int i = threadIdx.x; i < 64 * CHUNKS; i += AD_THREADS) {
             const int row = i / CHUNKS, c = i - row * CHUNKS;
             cp_async16(kb + tile_offset<D>(row, c), ks + (size_t)row * D + c * 8);
-            cp_async16(vb + tile_offset<D>(row, c), vs + (size_t)row * D + c * 8);
+            if (D == DV) cp_async16(vb + tile_offset<DV>(row, c), vs + (size_t)row * DV + c * 8);
         }
+        if (D != DV)
+            for (int i = threadIdx.x; i < 64 * VCHUNKS; i += AD_THREADS) {
+                const int row = i / VCHUNKS, c = i - row * VCHUNKS;
+                cp_async16(vb + tile_offset<DV>(row, c), vs + (size_t)row * DV + c * 8);
+            }
     };
 
     // The first pages are asked for at once, before the wait and before the query is fetched
@@ -302,7 +307,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             let_go();
             continue;
         }
-        const uint32_t kb = ad_smem(smem + (size_t)(it % AD_STAGES) * 2 * TILE_BYTES), vb = kb + TILE_BYTES;
+        const uint32_t kb = ad_smem(smem + (size_t)(it % AD_STAGES) * STAGE_BYTES), vb = kb + K_BYTES;
         const int key0 = 16 * warp;   // this warp's 16 positions of the page
         if (tile == end_tile - 1) {
             // The row's own page.  What lies past the row's position in it belongs to nobody (a
@@ -311,14 +316,14 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             // cleared in the copy.  And the block that appends puts the row itself there: its
             // key, rotated with the same four roundings as everywhere, and its value; the same
             // go to the cache for the steps to come.
-            uint8_t* kt = smem + (size_t)(it % AD_STAGES) * 2 * TILE_BYTES;
-            uint8_t* vt = kt + TILE_BYTES;
+            uint8_t* kt = smem + (size_t)(it % AD_STAGES) * STAGE_BYTES;
+            uint8_t* vt = kt + K_BYTES;
             const int pr = pos % BC_PAGE;
-            for (int i = threadIdx.x; i < (BC_PAGE - 1 - pr) * CHUNKS; i += AD_THREADS) {
-                const int row = pr + 1 + i / CHUNKS, c = i % CHUNKS;
-                *reinterpret_cast<uint4*>(vt + offset(row, c)) = make_uint4(0u, 0u, 0u, 0u);
+            for (int i = threadIdx.x; i < (BC_PAGE - 1 - pr) * VCHUNKS; i += AD_THREADS) {
+                const int row = pr + 1 + i / VCHUNKS, c = i % VCHUNKS;
+                *reinterpret_cast<uint4*>(vt + v_offset(row, c)) = make_uint4(0u, 0u, 0u, 0u);
             }
-            if (appends) {
+            if (D == DV && appends) {      // (the fused mode comes with values as wide as keys)
                 const int page = page_of(tile);
                 const bf16* kr = q + (size_t)r * q_stride + k_off + (size_t)g * D;
                 const bf16* vr = q + (size_t)r * q_stride + v_off + (size_t)g * D;
@@ -398,7 +403,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             o[nd + 1][0] *= c0; o[nd + 1][1] *= c0; o[nd + 1][2] *= c1; o[nd + 1][3] *= c1;
             uint32_t b0, b1, b2, b3;
             const int j = lane >> 3, rr = lane & 7;
-            ldmatrix_x4_trans(vb + offset(key0 + (j & 1) * 8 + rr, nd + (j >> 1)), b0, b1, b2, b3);
+            ldmatrix_x4_trans(vb + v_offset(key0 + (j & 1) * 8 + rr, nd + (j >> 1)), b0, b1, b2, b3);
             mma_16816(o[nd], pf, b0, b1);
             mma_16816(o[nd + 1], pf, b2, b3);
         }
@@ -416,9 +421,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // Merge the four warps (each saw other positions) in the order 0, 1, 2, 3.
     float* wm = reinterpret_cast<float*>(smem);              // [4][16] maxima
     float* wl = wm + 4 * 16;                                 // [4][16] sums
-    float* wo = wl + 4 * 16;                                 // [4][16][D] weighted values
-    float* po = wo + 4 * 16 * D;                             // [16][D] this block's merged sum, for its cluster peers
-    float* pm = po + 16 * D;                                 // [16] its maximum
+    float* wo = wl + 4 * 16;                                 // [4][16][DV] weighted values
+    float* po = wo + 4 * 16 * DV;                            // [16][DV] this block's merged sum, for its cluster peers
+    float* pm = po + 16 * DV;                                // [16] its maximum
     float* pl = pm + 16;                                     // [16] its normaliser
     if (tq == 0) {
         wm[warp * 16 + gq] = m0;
@@ -429,15 +434,15 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // Only the rows that are heads of the group are read below (4 of the tile's 16 with four heads a kv head): the others are not written.
 #pragma unroll
     for (int nd = 0; nd < ND; nd++) {
-        float* base = wo + (size_t)warp * 16 * D + nd * 8 + 2 * tq;
-        if (gq < group) *reinterpret_cast<float2*>(base + (size_t)gq * D) = make_float2(o[nd][0], o[nd][1]);
-        if (gq + 8 < group) *reinterpret_cast<float2*>(base + (size_t)(gq + 8) * D) = make_float2(o[nd][2], o[nd][3]);
+        float* base = wo + (size_t)warp * 16 * DV + nd * 8 + 2 * tq;
+        if (gq < group) *reinterpret_cast<float2*>(base + (size_t)gq * DV) = make_float2(o[nd][0], o[nd][1]);
+        if (gq + 8 < group) *reinterpret_cast<float2*>(base + (size_t)(gq + 8) * DV) = make_float2(o[nd][2], o[nd][3]);
     }
     ad_workers_sync();
-    // scratch: [row][head][split][D + 2]: the un-normalised sum, then maximum and normaliser.
-    const int stride = D + 2;
-    for (int i = threadIdx.x; i < group * D; i += AD_THREADS) {
-        const int hr = i / D, d = i - hr * D;
+    // scratch: [row][head][split][DV + 2]: the un-normalised sum, then maximum and normaliser.
+    const int stride = DV + 2;
+    for (int i = threadIdx.x; i < group * DV; i += AD_THREADS) {
+        const int hr = i / DV, d = i - hr * DV;
         float M = -INFINITY;
         for (int w = 0; w < 4; w++) M = fmaxf(M, wm[w * 16 + hr]);
         float L = 0.0f, O = 0.0f;
@@ -445,14 +450,14 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             const float mw = wm[w * 16 + hr];
             const float f = mw == -INFINITY ? 0.0f : exp2f(mw - M);
             L += wl[w * 16 + hr] * f;
-            O += wo[((size_t)w * 16 + hr) * D + d] * f;
+            O += wo[((size_t)w * 16 + hr) * DV + d] * f;
         }
         const int h = g * group + hr;
         if (n_splits == 1) {
             // A sink is one more position of score 0 that has no value: it adds 2^(0 - M) to the sum of the weights alone, once,
             // where a row's last sums are made (here and at the two merges below).
             if (sink && M != -INFINITY) L += exp2f(-M);
-            out[((size_t)r * H + h) * D + d] = __float2bfloat16_rn(L > 0.0f ? O * out_scale / L : 0.0f);
+            out[((size_t)r * H + h) * DV + d] = __float2bfloat16_rn(L > 0.0f ? O * out_scale / L : 0.0f);
         } else if (use_cluster) {
             po[i] = O;
             if (d == 0) {
@@ -463,8 +468,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             float* dst = scratch + (((size_t)r * H + h) * n_splits + split) * stride;
             __stcg(dst + d, O);
             if (d == 0) {
-                __stcg(dst + D, M);
-                __stcg(dst + D + 1, L);
+                __stcg(dst + DV, M);
+                __stcg(dst + DV + 1, L);
             }
         }
     }
@@ -484,7 +489,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         cl.sync();
         AD_STAMP(6);
         const int crank = split - part * csize;
-        const int total = group * D, share = (total + csize - 1) / csize;
+        const int total = group * DV, share = (total + csize - 1) / csize;
         // All reads of the peers' shared memory (a good tenth of a microsecond each) are asked
         // for before any is used; the splits are added in their order as ever.
         auto merge = [&](auto cap) {
@@ -494,13 +499,13 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
             for (int sp = 0; sp < CAP; sp++) ppo[sp] = cl.map_shared_rank(po, sp < csize ? sp : 0);
             for (int i = crank * share + threadIdx.x; i < min(total, (crank + 1) * share); i += AD_THREADS) {
-                const int hr = i / D, d = i - hr * D;
+                const int hr = i / DV, d = i - hr * DV;
                 float ms[CAP], ls[CAP], os[CAP];
 #pragma unroll
                 for (int sp = 0; sp < CAP; sp++) {
                     const bool has = sp < csize;
-                    ms[sp] = has ? ppo[sp][16 * D + hr] : -INFINITY;
-                    ls[sp] = has ? ppo[sp][16 * D + 16 + hr] : 0.0f;
+                    ms[sp] = has ? ppo[sp][16 * DV + hr] : -INFINITY;
+                    ls[sp] = has ? ppo[sp][16 * DV + 16 + hr] : 0.0f;
                     os[sp] = has ? ppo[sp][i] : 0.0f;
                 }
                 float M = -INFINITY;
@@ -515,13 +520,13 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 }
                 if (parts == 1) {
                     if (sink && M != -INFINITY) L += exp2f(-M);
-                    out[((size_t)r * H + g * group + hr) * D + d] = __float2bfloat16_rn(L > 0.0f ? O * out_scale / L : 0.0f);
+                    out[((size_t)r * H + g * group + hr) * DV + d] = __float2bfloat16_rn(L > 0.0f ? O * out_scale / L : 0.0f);
                 } else {
                     float* dst = scratch + (((size_t)r * H + g * group + hr) * parts + part) * stride;
                     __stcg(dst + d, O);
                     if (d == 0) {
-                        __stcg(dst + D, M);
-                        __stcg(dst + D + 1, L);
+                        __stcg(dst + DV, M);
+                        __stcg(dst + DV + 1, L);
                     }
                 }
             }
@@ -546,21 +551,21 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     ad_workers_sync();
     if (!is_last) return;
     __threadfence();
-    for (int i = threadIdx.x; i < group * D; i += AD_THREADS) {
-        const int hr = i / D, d = i - hr * D;
+    for (int i = threadIdx.x; i < group * DV; i += AD_THREADS) {
+        const int hr = i / DV, d = i - hr * DV;
         const int h = g * group + hr;
         const float* src = scratch + ((size_t)r * H + h) * parts * stride;
         float M = -INFINITY;
-        for (int sp = 0; sp < parts; sp++) M = fmaxf(M, __ldcg(src + (size_t)sp * stride + D));
+        for (int sp = 0; sp < parts; sp++) M = fmaxf(M, __ldcg(src + (size_t)sp * stride + DV));
         float L = 0.0f, O = 0.0f;
         for (int sp = 0; sp < parts; sp++) {
-            const float ms = __ldcg(src + (size_t)sp * stride + D);
+            const float ms = __ldcg(src + (size_t)sp * stride + DV);
             const float f = ms == -INFINITY ? 0.0f : exp2f(ms - M);
-            L += __ldcg(src + (size_t)sp * stride + D + 1) * f;
+            L += __ldcg(src + (size_t)sp * stride + DV + 1) * f;
             O += __ldcg(src + (size_t)sp * stride + d) * f;
         }
         if (sink && M != -INFINITY) L += exp2f(-M);
-        out[((size_t)r * H + h) * D + d] = __float2bfloat16_rn(L > 0.0f ? O * out_scale / L : 0.0f);
+        out[((size_t)r * H + h) * DV + d] = __float2bfloat16_rn(L > 0.0f ? O * out_scale / L : 0.0f);
     }
 }
 
@@ -584,16 +589,16 @@ extern "C" void bc_attention_decode_set_tma(int on) { g_ad_tma = on != 0; }
 static int g_ad_cluster16 = 1;
 extern "C" void bc_attention_decode_set_cluster16(int on) { g_ad_cluster16 = on != 0; }
 
-template <int D, bool TMA, bool BIAS>
+template <int D, int DV, bool TMA, bool BIAS>
 static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, int q_stride, const void* k_cache, const void* v_cache,
                      const int* page_table, const int* row_pos, const int* row_slot, void* out, float* scratch, int* counters, int rows, int H,
                      int G, int max_pages, int n_pages, int window, float scale, int n_splits, FusedRope fr, cudaStream_t s) {
-    constexpr int TILE_BYTES = 64 * D * 2;
-    constexpr int MERGE_BYTES = (2 * 4 * 16 + 4 * 16 * D + 16 * D + 32) * 4;
-    constexpr int SMEM = (AD_STAGES * 2 * TILE_BYTES > MERGE_BYTES ? AD_STAGES * 2 * TILE_BYTES : MERGE_BYTES) + 1024;
+    constexpr int STAGE_BYTES = 64 * (D + DV) * 2;
+    constexpr int MERGE_BYTES = (2 * 4 * 16 + 4 * 16 * DV + 16 * DV + 32) * 4;
+    constexpr int SMEM = (AD_STAGES * STAGE_BYTES > MERGE_BYTES ? AD_STAGES * STAGE_BYTES : MERGE_BYTES) + 1024;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, TMA, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, DV, TMA, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
         if (e != cudaSuccess) {
             bc_set_error("attention_decode: cannot set shared memory to %d: %s", SMEM, cudaGetErrorString(e));
             return (int)e;
@@ -612,7 +617,7 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
         static int sixteen = -1;
         if (sixteen < 0) {
             sixteen = 0;
-            if (cudaFuncSetAttribute(attention_decode_kernel<D, TMA, BIAS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
+            if (cudaFuncSetAttribute(attention_decode_kernel<D, DV, TMA, BIAS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
                 cudaLaunchConfig_t cfg = {};
                 cfg.gridDim = dim3(16, 1, 1);
                 cfg.blockDim = dim3(TMA ? AD_THREADS_TMA : AD_THREADS);
@@ -624,7 +629,7 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
                 cfg.attrs = attr;
                 cfg.numAttrs = 1;
                 int fit = 0;
-                if (cudaOccupancyMaxActiveClusters(&fit, attention_decode_kernel<D, TMA, BIAS>, &cfg) == cudaSuccess && fit > 0) sixteen = 1;
+                if (cudaOccupancyMaxActiveClusters(&fit, attention_decode_kernel<D, DV, TMA, BIAS>, &cfg) == cudaSuccess && fit > 0) sixteen = 1;
             }
             (void)cudaGetLastError();
         }
@@ -633,45 +638,50 @@ static int launch_as(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
     if (n_splits > 8 && csize < n_splits && !(scratch && counters)) csize = 1;
     const bool clustered = n_splits > 1 && fr.allow_cluster && csize > 1;
     if (clustered)
-        bc_launch_clustered(attention_decode_kernel<D, TMA, BIAS>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, dim3(csize, 1, 1), mk, mv, (const bf16*)q,
+        bc_launch_clustered(attention_decode_kernel<D, DV, TMA, BIAS>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, dim3(csize, 1, 1), mk, mv, (const bf16*)q,
                             q_stride, (const bf16*)k_cache, (const bf16*)v_cache, page_table, row_pos, row_slot, (bf16*)out, scratch, counters, H, G,
                             max_pages, n_pages, window, scale * 1.4426950408889634f, (const float2*)fr.cos_sin, fr.pairing, fr.fuse,
                             fr.k_off, fr.v_off, (bf16*)k_cache, (bf16*)v_cache, csize, fr.sink, fr.out_scale, fr.bias, fr.bias_reach);
     else
-        bc_launch(attention_decode_kernel<D, TMA, BIAS>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, mk, mv, (const bf16*)q, q_stride, (const bf16*)k_cache,
+        bc_launch(attention_decode_kernel<D, DV, TMA, BIAS>, grid, dim3(TMA ? AD_THREADS_TMA : AD_THREADS), (size_t)SMEM, s, mk, mv, (const bf16*)q, q_stride, (const bf16*)k_cache,
                   (const bf16*)v_cache, page_table, row_pos, row_slot, (bf16*)out, scratch, counters, H, G, max_pages, n_pages, window,
                   scale * 1.4426950408889634f, (const float2*)fr.cos_sin, fr.pairing, fr.fuse, fr.k_off, fr.v_off, (bf16*)k_cache,
                   (bf16*)v_cache, 0, fr.sink, fr.out_scale, fr.bias, fr.bias_reach);
     BC_LAUNCH_STATUS();
 }
 
-template <int D>
+template <int D, int DV>
 static int launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table, const int* row_pos,
                   const int* row_slot, void* out, float* scratch, int* counters, int rows, int H, int G, int max_pages, int n_pages,
                   int window, float scale, int n_splits, FusedRope fr, cudaStream_t s) {
     CUtensorMap mk = {}, mv = {};
-    if constexpr (D == 64 || D == 128) {
+    if constexpr ((D == 64 || D == 128) && (DV == 64 || DV == 128)) {
         // Pages by TMA: the cache as a matrix of [pages * kv heads * 64 positions, D], boxes of 64 x 64.
         if (g_ad_tma && bc_encode_tiled_fn() && (uintptr_t)k_cache % 16 == 0 && (uintptr_t)v_cache % 16 == 0) {
             const long long cache_rows = (long long)n_pages * G * BC_PAGE;
             int st = bc_cached_cache_map(&mk, k_cache, cache_rows, D, "attention_decode");
-            if (st == BC_OK) st = bc_cached_cache_map(&mv, v_cache, cache_rows, D, "attention_decode");
+            if (st == BC_OK) st = bc_cached_cache_map(&mv, v_cache, cache_rows, DV, "attention_decode");
             if (st != BC_OK) return st;
-            return fr.bias ? launch_as<D, true, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H,
+            return fr.bias ? launch_as<D, DV, true, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H,
                                                       G, max_pages, n_pages, window, scale, n_splits, fr, s)
-                           : launch_as<D, true, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H,
+                           : launch_as<D, DV, true, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H,
                                                        G, max_pages, n_pages, window, scale, n_splits, fr, s);
         }
     }
-    return fr.bias ? launch_as<D, false, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
+    return fr.bias ? launch_as<D, DV, false, true>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
                                                max_pages, n_pages, window, scale, n_splits, fr, s)
-                   : launch_as<D, false, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
+                   : launch_as<D, DV, false, false>(mk, mv, q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G,
                                                 max_pages, n_pages, window, scale, n_splits, fr, s);
 }
 
 // Whether this kernel takes the sizes (else the caller uses the one-warp-a-row kernel).
 extern "C" int bc_attention_decode_accepts(int H, int G, int D) {
     return G > 0 && H % G == 0 && H / G <= AD_MAX_GROUP && D % 16 == 0 && D >= 16 && D <= 128;
+}
+
+// The same with values DV wide: DV = D, or one of these pairs.
+extern "C" int bc_attention_decode_accepts_kv(int H, int G, int D, int DV) {
+    return bc_attention_decode_accepts(H, G, D) && (D == DV || (D == 64 && (DV == 32 || DV == 128)) || (D == 128 && (DV == 32 || DV == 64)) || (D == 32 && DV == 64));
 }
 
 // Floats of scratch and ints of counters for `rows` rows cut into `n_splits`.
@@ -689,13 +699,14 @@ extern "C" int bc_attention_decode_workspace(int rows, int H, int G, int D, int 
 // null for no rotation.  Two to eight splits run as a thread-block cluster and need no
 // scratch memory; adding 4 to fuse sends them through scratch memory like larger counts.
 static int decode_fused(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table, const int* row_pos,
-                        const int* row_slot, void* out, float* scratch, int* counters, int rows, int H, int G, int D, int max_pages, int n_pages,
+                        const int* row_slot, void* out, float* scratch, int* counters, int rows, int H, int G, int D, int DV, int max_pages, int n_pages,
                         int window, float scale, int n_splits, const float* cos_sin, int pairing, int fuse, int sink, float out_scale,
                         const float* bias, int bias_reach, cudaStream_t s) {
     BC_CHECK_ARG(bias == nullptr || bias_reach > 0, "attention_decode: a table of biases for %d distances", bias_reach);
     BC_CHECK_ARG(rows >= 0 && rows <= 65535, "attention_decode: %d rows (at most 65535)", rows);
-    BC_CHECK_ARG(bc_attention_decode_accepts(H, G, D), "attention_decode: H=%d G=%d D=%d is outside what this kernel takes "
-                 "(at most %d heads a kv head, head size a multiple of 16 up to 128)", H, G, D, AD_MAX_GROUP);
+    BC_CHECK_ARG(bc_attention_decode_accepts_kv(H, G, D, DV), "attention_decode: H=%d G=%d D=%d DV=%d is outside what this kernel takes "
+                 "(at most %d heads a kv head, head size a multiple of 16 up to 128, a few other widths of values)", H, G, D, DV, AD_MAX_GROUP);
+    BC_CHECK_ARG((fuse & 3) == 0 || D == DV, "attention_decode: the fused mode takes values as wide as keys");
     BC_CHECK_ARG(n_splits >= 1 && n_splits <= 65535 && G <= 65535, "attention_decode: bad split count %d", n_splits);
     BC_CHECK_ARG(n_splits == 1 || (n_splits <= 8 && (fuse & 4) == 0) || (scratch && counters), "attention_decode: these splits need scratch memory");
     BC_CHECK_ARG(q_stride % 2 == 0 && ((uintptr_t)q % 4 == 0), "attention_decode: q must be 4-byte aligned with an even stride");
@@ -704,8 +715,12 @@ static int decode_fused(const void* q, int q_stride, const void* k_cache, const 
     BC_CHECK_ARG((fuse & 3) == 0 || cos_sin == nullptr || (uintptr_t)cos_sin % 16 == 0, "attention_decode: the rotary table must be 16-byte aligned");
     if (rows == 0) return BC_OK;
     FusedRope fr{cos_sin, pairing, fuse & 3, H * D, (H + G) * D, (fuse & 4) == 0, sink, out_scale, bias, bias_reach};
+#define AD_PAIR(DD, VV) \
+    if (D == DD && DV == VV) return launch<DD, VV>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, max_pages, n_pages, window, scale, n_splits, fr, s);
+    AD_PAIR(64, 32) AD_PAIR(64, 128) AD_PAIR(128, 32) AD_PAIR(128, 64) AD_PAIR(32, 64)
+#undef AD_PAIR
 #define AD_CASE(DD) \
-    case DD: return launch<DD>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, max_pages, n_pages, window, scale, n_splits, fr, s);
+    case DD: return launch<DD, DD>(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, max_pages, n_pages, window, scale, n_splits, fr, s);
     switch (D) {
         AD_CASE(16) AD_CASE(32) AD_CASE(48) AD_CASE(64) AD_CASE(80) AD_CASE(96) AD_CASE(112) AD_CASE(128)
     }
@@ -718,19 +733,19 @@ extern "C" int bc_attention_decode_fused_bf16(const void* q, int q_stride, const
                                               const int* row_pos, const int* row_slot, void* out, float* scratch, int* counters, int rows,
                                               int H, int G, int D, int max_pages, int n_pages, int window, float scale, int n_splits,
                                               const float* cos_sin, int pairing, int fuse, cudaStream_t s) {
-    return decode_fused(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, D, max_pages, n_pages, window,
+    return decode_fused(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, D, D, max_pages, n_pages, window,
                         scale, n_splits, cos_sin, pairing, fuse, 0, 1.0f, nullptr, 0, s);
 }
 
 // The plain kernel (q rotated already, the cache holding the row) with a sink (one more position of score 0 without a value,
-// counted once where a row's last sums are made), a factor on the output and biases by distance (a table as in common.cuh, in log2
+// counted once where a row's last sums are made), a factor on the output, values DV wide (out: [rows, H DV]; scratch for DV) and biases by distance (a table as in common.cuh, in log2
 // units, or null); fuse: 0, or 4 to send the splits through scratch.
 extern "C" int bc_attention_decode_sink_bf16(const void* q, int q_stride, const void* k_cache, const void* v_cache, const int* page_table,
                                              const int* row_pos, const int* row_slot, void* out, float* scratch, int* counters, int rows,
-                                             int H, int G, int D, int max_pages, int n_pages, int window, float scale, int n_splits, int fuse,
+                                             int H, int G, int D, int DV, int max_pages, int n_pages, int window, float scale, int n_splits, int fuse,
                                              int sink, float out_scale, const float* bias, int bias_reach, cudaStream_t s) {
     BC_CHECK_ARG((fuse & 3) == 0, "attention_decode: the sink comes with the plain kernel (fuse %d)", fuse);
-    return decode_fused(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, D, max_pages, n_pages, window,
+    return decode_fused(q, q_stride, k_cache, v_cache, page_table, row_pos, row_slot, out, scratch, counters, rows, H, G, D, DV, max_pages, n_pages, window,
                         scale, n_splits, nullptr, 0, fuse, sink, out_scale, bias, bias_reach, s);
 }
 
@@ -776,7 +791,7 @@ static int launch_static(float* scratch, int* counters, const void* q, int q_str
         // First call for this head size on this device: let the kernel use the shared memory it needs.
         std::lock_guard<std::mutex> lock(g_static_mutex);
         if (!(g_static_configured[device] & (1u << (D / 16)))) {
-            cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+            cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D, D, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
             if (e != cudaSuccess) {
                 bc_set_error("attention_decode_static: cannot set shared memory to %d: %s", SMEM, cudaGetErrorString(e));
                 return (int)e;
@@ -784,7 +799,7 @@ static int launch_static(float* scratch, int* counters, const void* q, int q_str
             g_static_configured[device] |= 1u << (D / 16);
         }
     }
-    bc_launch(attention_decode_kernel<D, false, false>, dim3(n_splits, G, rows), dim3(AD_THREADS), (size_t)SMEM, s, none, none, (const bf16*)q, q_stride,
+    bc_launch(attention_decode_kernel<D, D, false, false>, dim3(n_splits, G, rows), dim3(AD_THREADS), (size_t)SMEM, s, none, none, (const bf16*)q, q_stride,
               (const bf16*)k_cache, (const bf16*)v_cache, page_table, row_pos, row_slot, (bf16*)out, scratch, counters, H, G, max_pages,
               n_pages, window, scale * 1.4426950408889634f, (const float2*)nullptr, 0, 0, 0, 0, (bf16*)nullptr, (bf16*)nullptr, 0, 0, 1.0f, (const float*)nullptr, 0);
     BC_LAUNCH_STATUS();

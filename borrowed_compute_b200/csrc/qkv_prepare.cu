@@ -191,7 +191,17 @@ extern "C" int bc_qkv_prepare_bf16(const float* qkv, const float* bias, const fl
 // take pairs of dimensions, so the sum of squares and the rotation need no second pass over memory; which
 // values a lane adds, and in which order, depends on the sizes alone.  Values may have a number of heads of their own (VG: two
 // key maps that share one value head, say), and a layer that reads another layer's cache projects queries alone (G = VG = 0).
-template <class T>
+// VEC: nothing turns and every width is a multiple of four, so that a lane takes four neighbouring dimensions at a time.
+template <class T> __device__ __forceinline__ void prepare_store4(T* p, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void prepare_store4<float>(float* p, float a, float b, float c, float d) {
+    *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+template <> __device__ __forceinline__ void prepare_store4<bf16>(bf16* p, float a, float b, float c, float d) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+}
+
+template <class T, bool VEC>
 __global__ void __launch_bounds__(256)
 qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                          const float* __restrict__ cos_sin, int n_positions, const int* __restrict__ row_pos, const int* __restrict__ row_slot,
@@ -223,7 +233,14 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
         const float* wt = is_q ? q_weight : k_weight;
         float ss = 0.0f;
         if (normed) {
-            for (int d = lane; d < D; d += 32) ss = fmaf(xh[d], xh[d], ss);
+            if (VEC) {
+                for (int d = 4 * lane; d < D; d += 128) {
+                    const float4 v = *reinterpret_cast<const float4*>(xh + d);      // again below: by then in the L1
+                    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+                }
+            } else {
+                for (int d = lane; d < D; d += 32) ss = fmaf(xh[d], xh[d], ss);
+            }
             ss = warp_sum(ss);
         }
         const float scale = normed ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
@@ -231,6 +248,15 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
         T* dst = is_q ? q_out + (size_t)r * nq + (size_t)head * D
                       : k_cache + (((size_t)(cache ? page : 0) * G + (head - H)) * BC_PAGE + pos % BC_PAGE) * D;
         if (!is_q && !cache) continue;
+        if (VEC) {
+            for (int d = 4 * lane; d < D; d += 128) {
+                const float4 v = *reinterpret_cast<const float4*>(xh + d);
+                const float4 w = normed ? *reinterpret_cast<const float4*>(wt + d) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+                const float f = scale * more;
+                prepare_store4<T>(dst + d, v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w);
+            }
+            continue;
+        }
         for (int u = lane; u < units; u += 32) {
             if (u < half) {
                 const int a = pairing ? 2 * u : u, b = pairing ? 2 * u + 1 : u + half;
@@ -249,7 +275,13 @@ qkv_prepare_heads_kernel(const float* __restrict__ qkv, const float* __restrict_
             }
         }
     }
-    if (cache) {
+    if (cache && VEC) {
+        for (int i = 4 * threadIdx.x; i < nv; i += 4 * blockDim.x) {
+            const int g = i / DV, d = i - g * DV;
+            const float4 v = *reinterpret_cast<const float4*>(x + nq + nk + i);
+            prepare_store4<T>(v_cache + (((size_t)page * VG + g) * BC_PAGE + pos % BC_PAGE) * DV + d, v.x, v.y, v.z, v.w);
+        }
+    } else if (cache) {
         for (int i = threadIdx.x; i < nv; i += blockDim.x) {
             const int g = i / DV, d = i - g * DV;
             v_cache[(((size_t)page * VG + g) * BC_PAGE + pos % BC_PAGE) * DV + d] = from_f32<T>(x[nq + nk + i]);
@@ -268,7 +300,9 @@ static int launch_heads(const float* qkv, const float* q_weight, const float* k_
     if (rows == 0) return BC_OK;
     const int heads = H + G;
     const int threads = heads >= 8 ? 256 : heads >= 4 ? 128 : 64;      // by the row's heads alone
-    bc_launch(qkv_prepare_heads_kernel<T>, dim3(rows), dim3(threads), 0, s, qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot,
+    const bool vec = rot == 0 && D % 4 == 0 && DV % 4 == 0 && (uintptr_t)qkv % 16 == 0 && (uintptr_t)q_weight % 16 == 0 && (uintptr_t)k_weight % 16 == 0 &&
+                     (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_cache % 16 == 0 && (uintptr_t)v_cache % 16 == 0;
+    bc_launch(vec ? qkv_prepare_heads_kernel<T, true> : qkv_prepare_heads_kernel<T, false>, dim3(rows), dim3(threads), 0, s, qkv, q_weight, k_weight, cos_sin, n_positions, row_pos, row_slot,
               page_table, max_pages, n_pages, (T*)q_out, (T*)k_cache, (T*)v_cache, H, G, VG, D, DV, rot, pairing, eps, normed, write_cache, temp_coef, temp_every);
     BC_LAUNCH_STATUS();
 }

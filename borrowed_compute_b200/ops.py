@@ -1857,10 +1857,11 @@ def set_attention_decode_cluster16(on: bool) -> None:
     lib().bc_attention_decode_set_cluster16(_c_int(1 if on else 0))
 
 
-def attention_decode_accepts(heads: int, kv_heads: int, head_dim: int, dtype: torch.dtype) -> bool:
+def attention_decode_accepts(heads: int, kv_heads: int, head_dim: int, dtype: torch.dtype, value_dim: Optional[int] = None) -> bool:
     """Whether the split decode kernel takes these sizes (bf16; at most 16 heads a kv head;
-    head size a multiple of 16 up to 128).  Otherwise attention_rows serves."""
-    return dtype == torch.bfloat16 and bool(_fn("bc_attention_decode_accepts")(_c_int(heads), _c_int(kv_heads), _c_int(head_dim)))
+    head size a multiple of 16 up to 128; values as wide as keys, or a few pairs of widths).  Otherwise attention_rows serves."""
+    return dtype == torch.bfloat16 and bool(_fn("bc_attention_decode_accepts_kv")(_c_int(heads), _c_int(kv_heads), _c_int(head_dim),
+                                                                                 _c_int(head_dim if value_dim is None else value_dim)))
 
 
 def attention_decode_splits(rows: int, kv_heads: int, max_pages: int) -> int:
@@ -1909,7 +1910,8 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
                      row_pos: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                      window: int = 0, scale: Optional[float] = None, splits: Optional[int] = None, fuse: int = 0,
                      cos_sin: Optional[torch.Tensor] = None, pairing: int = 0, via_scratch: bool = False,
-                     reach: Optional[int] = None, sink: bool = False, out_scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
+                     reach: Optional[int] = None, sink: bool = False, out_scale: float = 1.0, bias: Optional[torch.Tensor] = None,
+                     value_dim: Optional[int] = None) -> None:
     """Attention of one new row a sequence (bf16): the cached positions are split across
     blocks and the heads of a kv head share each read; results are merged in a fixed order.
     Two to eight splits form a thread-block cluster and merge through one another's shared
@@ -1920,7 +1922,9 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
     a bound on the positions any row reaches (else what the page table can hold); the
     number of splits is chosen by it, no result depends on it.  ``sink`` adds one to the softmax's
     denominator (a position of score 0 without a value), ``out_scale`` multiplies the result, ``bias``
-    (biases by distance, ``parts/distance_bias.py``, in log2 units) is added to the scores: all three with the plain kernel (``fuse`` 0) only."""
+    (biases by distance, ``parts/distance_bias.py``, in log2 units) is added to the scores, ``value_dim`` (default: ``head_dim``) is the
+    width of a head's values: these with the plain kernel (``fuse`` 0) only."""
+    value_dim = head_dim if value_dim is None else int(value_dim)
     _need(q, "q", torch.bfloat16)
     _need(k_cache, "k_cache", torch.bfloat16)
     _need(v_cache, "v_cache", torch.bfloat16)
@@ -1929,10 +1933,11 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
     _need(row_slot, "row_slot", torch.int32)
     _need(out, "out", torch.bfloat16)
     rows = out.shape[0]
-    if out.shape[1] != heads * head_dim:
-        raise KernelError(f"attention: out width {out.shape[1]} is not heads * head_dim")
-    if tuple(k_cache.shape[1:]) != (kv_heads, PAGE, head_dim) or k_cache.shape != v_cache.shape:
-        raise KernelError(f"attention: cache is {tuple(k_cache.shape)}, wanted [pages, {kv_heads}, {PAGE}, {head_dim}]")
+    if out.shape[1] != heads * value_dim:
+        raise KernelError(f"attention: out width {out.shape[1]} is not heads * value_dim")
+    if tuple(k_cache.shape[1:]) != (kv_heads, PAGE, head_dim) or tuple(v_cache.shape) != tuple(k_cache.shape[:3]) + (value_dim,):
+        raise KernelError(f"attention: cache is {tuple(k_cache.shape)} and {tuple(v_cache.shape)}, wanted [pages, {kv_heads}, {PAGE}, {head_dim}] "
+                          f"and values {value_dim} wide")
     if scale is None:
         scale = 1.0 / float(head_dim) ** 0.5
     if splits is None:
@@ -1944,7 +1949,7 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
         splits = attention_decode_splits(rows, kv_heads, pages)
     scratch = counters = None
     if splits > 1:
-        scratch, counters = _decode_workspace(q.device, rows * heads * splits * (head_dim + 2), rows * kv_heads)
+        scratch, counters = _decode_workspace(q.device, rows * heads * splits * (value_dim + 2), rows * kv_heads)
     if cos_sin is not None:
         _need(cos_sin, "cos_sin", torch.float32)
         if tuple(cos_sin.shape[1:]) != (head_dim // 2, 2):
@@ -1952,12 +1957,12 @@ def attention_decode(q: torch.Tensor, q_stride: int, k_cache: torch.Tensor, v_ca
         if bounds_check and not torch.cuda.is_current_stream_capturing():
             _bounds("attention_decode: row_pos (against the rotary table)", row_pos.reshape(-1)[:rows][row_slot.reshape(-1)[:rows] >= 0], cos_sin.shape[0])
     _bounds_paged("attention_decode", rows, row_pos, row_slot, page_table, k_cache.shape[0])
-    if sink or out_scale != 1.0 or bias is not None:
+    if sink or out_scale != 1.0 or bias is not None or value_dim != head_dim:
         if fuse != 0:
-            raise KernelError("attention_decode: a sink, biases or a factor comes with the plain kernel (fuse 0)")
+            raise KernelError("attention_decode: a sink, biases, values of their own width or a factor comes with the plain kernel (fuse 0)")
         _call(_fn("bc_attention_decode_sink_bf16"), _ptr(q), _c_int(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _ptr(row_pos),
               _ptr(row_slot), _ptr(out), _ptr(scratch), _ptr(counters), _c_int(rows), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
-              _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_float(scale), _c_int(splits),
+              _c_int(value_dim), _c_int(page_table.shape[1]), _c_int(k_cache.shape[0]), _c_int(window), _c_float(scale), _c_int(splits),
               _c_int(4 if via_scratch else 0), _c_int(1 if sink else 0), _c_float(out_scale), _ptr(bias),
               _c_int(_bias_reach(bias, heads, kv_heads, "attention_decode")), _stream())
         return

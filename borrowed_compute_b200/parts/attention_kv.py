@@ -136,10 +136,11 @@ class GroupedQueryAttentionKV(Mixer):
                                   ctx.seqs, ctx.max_new, H, G, D, window=self.window, scale=self.scale, use_tc=True, chunk=self.chunk,
                                   value_dim=DV, sink=self.sink, out_scale=self.out_scale, bias=self.bias_log2)
             return
-        if not force_rows and not force_tiles and ctx.decode and D == DV and self.chunk == 0 and ops.attention_decode_accepts(H, G, D, q.dtype):
-            # Single rows over keys and values of one width, no chunk mask: the kernel that splits a row's positions over blocks.
+        if not force_rows and not force_tiles and ctx.decode and self.chunk == 0 and ops.attention_decode_accepts(H, G, D, q.dtype, DV):
+            # Single rows without a chunk mask: the kernel that splits a row's positions over blocks.
             ops.attention_decode(q, H * D, mem.k_pages, mem.v_pages, mem.page_table, ctx.row_pos, ctx.row_slot, out, H, G, D, window=self.window,
-                                 scale=self.scale, reach=ctx.max_total, sink=self.sink, out_scale=self.out_scale, bias=self.bias_log2)
+                                 scale=self.scale, reach=ctx.max_total, sink=self.sink, out_scale=self.out_scale, bias=self.bias_log2,
+                                 value_dim=DV)
             return
         if not force_rows and ops.attention_tiles_accepts(H, G, D, DV, q.dtype):
             # Tensor-core tiles, for prompts and for single rows alike: the heads of a kv head share every page read.
