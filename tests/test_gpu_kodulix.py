@@ -49,7 +49,7 @@ def scores_close(got, ref, clear, dtype, what=""):
     assert got.shape == ref.shape and np.isfinite(got).all(), f"{what}: shape or numbers"
     off = np.sqrt(((got - ref) ** 2).mean(axis=-1)) / ref.std()
     mine = off[clear] if clear.any() else off
-    assert np.median(mine) <= 0.03 and np.quantile(mine, 0.9) <= 0.12, \
+    assert np.median(mine) <= 0.02 and np.quantile(mine, 0.9) <= 0.08, \
         f"{what}: of {mine.size} clear rows the median is off by {np.median(mine):.4g}, the 90th percentile by {np.quantile(mine, 0.9):.4g} of the spread"
 
 
