@@ -33,6 +33,8 @@
 // the second query tile) are the softmax and write the output.  Every wait is bounded
 // (about a second); a wait that gives up records where in a status word, and the block
 // frees its TMEM and returns.
+#include <type_traits>
+
 #include "mma_tiles.cuh"
 #include "tc_ptx.cuh"
 #include "tma_host.cuh"
@@ -302,11 +304,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const bool near = BIAS && warp_first_pos - (tile * BC_PAGE + BC_PAGE - 1) < bias_reach - 1;
             if (BIAS && near) {
                 const float* bp = my_bias + (ptrdiff_t)max(pos - tile * BC_PAGE, 0) * group;      // position 0 of the page; then one distance nearer each
+                // The usual group sizes as constants: the loads then differ in their immediate offsets alone.
+                auto add_bias = [&](auto heads) {
+                    constexpr int HEADS = decltype(heads)::value;
 #pragma unroll
-                for (int c = 0; c < 64; c++) {
-                    sv[c] = __float_as_uint(fmaf(__uint_as_float(sv[c]), scale_log2, __ldg(bp)));
-                    bp -= group;
-                }
+                    for (int c = 0; c < 64; c++) {
+                        sv[c] = __float_as_uint(fmaf(__uint_as_float(sv[c]), scale_log2, __ldg(HEADS ? bp - c * HEADS : bp)));
+                        if (!HEADS) bp -= group;
+                    }
+                };
+                if (group == 4) add_bias(std::integral_constant<int, 4>());
+                else if (group == 8) add_bias(std::integral_constant<int, 8>());
+                else add_bias(std::integral_constant<int, 0>());
             }
             const float page_scale = BIAS && near ? 1.0f : scale_log2, page_bias = BIAS && !near ? far_bias : 0.0f;
             if (whole) {
